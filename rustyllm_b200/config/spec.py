@@ -109,6 +109,7 @@ class ModelSpec:
     ignored_tensors: Tuple[str, ...] = ()  # names that may be in the file and are not read
     inject_parts: Tuple[PartSpec, ...] = ()      # parts of role "inject" (parts/inject.py)
     injections: Tuple[Injection, ...] = ()       # where along the schedule they act, in running order
+    streams: int = 0                     # a residual of this many streams (parts/streams.py); 0: one plain residual
 
     def validate(self) -> None:
         n = len(self.layers)
@@ -116,6 +117,10 @@ class ModelSpec:
             raise ValueError("a model needs at least one layer")
         if not self.schedule:
             raise ValueError("the schedule of layers is empty")
+        if self.streams < 0:
+            raise ValueError(f"streams must be >= 0, got {self.streams}")
+        if self.streams and self.injections:
+            raise ValueError("additions between layers on a residual of several streams are not built")
         for i in self.schedule:
             if not (0 <= i < n):
                 raise ValueError(f"schedule names layer {i}, but there are {n} layers")

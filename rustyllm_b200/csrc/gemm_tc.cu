@@ -132,7 +132,7 @@ __device__ __forceinline__ void tile_epilogue(uint32_t tmem_acc, int quarter, in
         const float got = __shfl_xor_sync(0xffffffffu, even ? hi : lo, 1);
         const float gate = even ? lo : got, up = even ? got : hi;
         const int m = m0 + c * 16 + (even ? j : j + 8);
-        if ((n | 1) < N && m < M) ob[(size_t)m * ldo + (n >> 1)] = __float2bfloat16_rn(gated_mul(gate, up, out_mode));
+        if ((n | 1) < N && m < M) ob[(size_t)m * ldo + (n >> 1)] = __float2bfloat16_rn(gated_mul(gate, up, out_mode, fuse.act_limit, fuse.act_alpha));
       }
     } else if (out_mode == TC_OUT_ADD_F32) {
       // all sixteen loads of the residual first, then the stores: a load placed after
@@ -433,7 +433,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
                           const __grid_constant__ CUtensorMap map_a_tail, const float* __restrict__ bias,
                           void* __restrict__ out, int out_mode, int M, int N, int K,
                           int ldo, int* __restrict__ err, int tiles_m, int num_tiles, const TcTail tail,
-                          const int* __restrict__ tile_group, int group_rows) {
+                          const int* __restrict__ tile_group, int group_rows, float act_limit, float act_alpha) {
   // tile_group (null: none): the weight is stacked matrices of group_rows rows, and the token tile of BT rows at
   // m0 multiplies with matrix tile_group[m0 / BT]; negative: the tile is skipped by every role alike.  The table
   // is written by a kernel in front, so each role reads it behind its wait.
@@ -563,8 +563,11 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
         break;
       }
       tc_fence_after();
+      TcFuse fuse = {};
+      fuse.act_limit = act_limit;
+      fuse.act_alpha = act_alpha;
       tile_epilogue<BT>(tmem_base + (uint32_t)(buf * BT), quarter, lane, at.n0, at.m0, min(at.bt, M - at.m0), M, N, ldo, bias, out,
-                        out_mode, TcFuse{}, nullptr);
+                        out_mode, fuse, nullptr);
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&acc_empty[buf]));    // this warp has read the accumulator
@@ -580,7 +583,9 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
 template <int BT>
 static int launch_tc_persistent(const CUtensorMap& mw, const CUtensorMap& ma, const void* A, int lda, const float* bias,
                                 void* out, int out_mode, int M, int N, int K, int ldo, int* err, cudaStream_t stream,
-                                const int* tile_group = nullptr, int group_rows = 0) {
+                                const TcFuse& fuse) {
+  const int* tile_group = fuse.tile_group;
+  const int group_rows = fuse.group_rows;
   using Cfg = TcConfig<BT>;
   static bool configured = false;
   if (!configured) {
@@ -616,7 +621,8 @@ static int launch_tc_persistent(const CUtensorMap& mw, const CUtensorMap& ma, co
   }
   const int grid = num_tiles < num_sms ? num_tiles : num_sms;
   cudaError_t e = rl_launch_pdl(gemm_tc_persistent_kernel<BT>, dim3(grid), dim3(TC_THREADS), (size_t)Cfg::SMEM_BYTES, stream,
-                                mw, ma, ma_tail, bias, out, out_mode, M, N, K, ldo, err, tiles_m, num_tiles, tail, tile_group, group_rows);
+                                mw, ma, ma_tail, bias, out, out_mode, M, N, K, ldo, err, tiles_m, num_tiles, tail, tile_group, group_rows,
+                                fuse.act_limit, fuse.act_alpha);
   if (e != cudaSuccess) {
     rl_set_error("rl_gemm_tc: launch of the persistent kernel failed: %s", cudaGetErrorString(e));
     return RL_ERR_CUDA;
@@ -787,7 +793,7 @@ static int gemm_tc_run(const void* A, const void* W, const float* bias, void* ou
   const float* norm_weight = fuse.norm_weight;
   RL_REQUIRE(rl_gemm_tc_supported(A, W, M, N, K, lda), "rl_gemm_tc: operands not supported (M=%d N=%d K=%d lda=%d; K and lda "
              "must be multiples of 8 and the bases 16-byte aligned)", M, N, K, lda);
-  RL_REQUIRE(out_mode >= 0 && out_mode <= 6, "rl_gemm_tc: unknown output mode %d", out_mode);
+  RL_REQUIRE(out_mode >= 0 && out_mode <= 7, "rl_gemm_tc: unknown output mode %d", out_mode);
   RL_REQUIRE(!tc_out_gated(out_mode) || N % 2 == 0, "rl_gemm_tc: the SwiGLU epilogue needs an even number of weight rows, got %d", N);
   RL_REQUIRE(ldo >= (tc_out_gated(out_mode) ? N / 2 : N) && err != nullptr, "rl_gemm_tc: bad output stride or null error word");
   RL_REQUIRE(force_splits >= 0 && force_splits <= 8, "rl_gemm_tc: the number of K parts must be 1 to 8 (0: chosen from the shapes), got %d", force_splits);
@@ -821,40 +827,53 @@ static int gemm_tc_run(const void* A, const void* W, const float* bias, void* ou
     if (bt == 128) return launch_tc<128>(mw, ma, bias, out, out_mode, M, N, K, ldo, err, splits, kb_per, fuse, stream);
     return launch_tc<256>(mw, ma, bias, out, out_mode, M, N, K, ldo, err, splits, kb_per, fuse, stream);
   }
-  if (bt == 128) return launch_tc_persistent<128>(mw, ma, A, lda, bias, out, out_mode, M, N, K, ldo, err, stream);
-  return launch_tc_persistent<256>(mw, ma, A, lda, bias, out, out_mode, M, N, K, ldo, err, stream);
+  if (bt == 128) return launch_tc_persistent<128>(mw, ma, A, lda, bias, out, out_mode, M, N, K, ldo, err, stream, fuse);
+  return launch_tc_persistent<256>(mw, ma, A, lda, bias, out, out_mode, M, N, K, ldo, err, stream, fuse);
 }
 
-extern "C" int rl_gemm_tc(const void* A, const void* W, const float* bias, void* out, int out_mode, int M, int N,
-                          int K, int lda, int ldo, int* err, int force_splits, const float* scale_partials,
-                          int scale_count, float scale_eps, const float* norm_weight, void* norm_out, int ld_norm,
-                          float* norm_partials, cudaStream_t stream) {
+// act_limit, act_alpha: the constants of out_mode 7 (else unused)
+extern "C" int rl_gemm_tc_act(const void* A, const void* W, const float* bias, void* out, int out_mode, int M, int N,
+                              int K, int lda, int ldo, int* err, int force_splits, const float* scale_partials,
+                              int scale_count, float scale_eps, const float* norm_weight, void* norm_out, int ld_norm,
+                              float* norm_partials, float act_limit, float act_alpha, cudaStream_t stream) {
   RL_REQUIRE(out_mode != TC_OUT_ROPE_KV, "rl_gemm_tc: the rotation epilogue has its own entry point, rl_gemm_tc_qkv_rope");
   TcFuse fuse = {};
+  fuse.act_limit = act_limit; fuse.act_alpha = act_alpha;
   fuse.scale_partials = scale_partials; fuse.scale_count = scale_count; fuse.scale_eps = scale_eps;
   fuse.norm_weight = norm_weight; fuse.norm_out = (__nv_bfloat16*)norm_out; fuse.ld_norm = ld_norm;
   fuse.norm_partials = norm_partials;
   return gemm_tc_run(A, W, bias, out, out_mode, M, N, K, lda, ldo, err, force_splits, fuse, stream);
 }
 
+extern "C" int rl_gemm_tc(const void* A, const void* W, const float* bias, void* out, int out_mode, int M, int N,
+                          int K, int lda, int ldo, int* err, int force_splits, const float* scale_partials,
+                          int scale_count, float scale_eps, const float* norm_weight, void* norm_out, int ld_norm,
+                          float* norm_partials, cudaStream_t stream) {
+  RL_REQUIRE(out_mode != TC_OUT_CLAMPED, "rl_gemm_tc: the clamped gate takes its constants through rl_gemm_tc_act");
+  return rl_gemm_tc_act(A, W, bias, out, out_mode, M, N, K, lda, ldo, err, force_splits, scale_partials, scale_count, scale_eps,
+                        norm_weight, norm_out, ld_norm, norm_partials, 0.f, 0.f, stream);
+}
+
 // Grouped product: W is `groups` matrices [N, K] one after another ([groups * N, K]); token tile t (rows
 // t * bt .. of A and of out) multiplies with matrix tile_group[t] (device ints, written by a kernel in front;
 // negative: the tile is skipped and its rows of out stay as they are).  A: [M, K] with M a multiple of the
 // token tile bt (16, 32, 64, 128 or 256), rows ordered by group and padded so that no tile holds two groups.
-// out_mode 0, 1, 2 or 3 as in rl_gemm_tc; no bias, no norm riding along.
+// out_mode 0, 1, 2, 3 or (act_limit, act_alpha) 7 as in rl_gemm_tc; no bias, no norm riding along.
 extern "C" int rl_gemm_tc_grouped(const void* A, const void* W, void* out, int out_mode, int M, int N, int K, int lda,
-                                  int ldo, int* err, const int* tile_group, int groups, int bt, cudaStream_t stream) {
+                                  int ldo, int* err, const int* tile_group, int groups, int bt, float act_limit, float act_alpha,
+                                  cudaStream_t stream) {
   RL_REQUIRE(rl_gemm_tc_supported(A, W, M, N, K, lda), "rl_gemm_tc_grouped: operands not supported (M=%d N=%d K=%d lda=%d; K and lda "
              "must be multiples of 8 and the bases 16-byte aligned)", M, N, K, lda);
-  RL_REQUIRE(out_mode >= 0 && out_mode <= 3, "rl_gemm_tc_grouped: unknown output mode %d", out_mode);
-  RL_REQUIRE(out_mode != TC_OUT_SWIGLU || N % 2 == 0, "rl_gemm_tc_grouped: the SwiGLU epilogue needs an even number of weight rows, got %d", N);
-  RL_REQUIRE(ldo >= (out_mode == TC_OUT_SWIGLU ? N / 2 : N) && err != nullptr && tile_group != nullptr && groups > 0,
+  RL_REQUIRE((out_mode >= 0 && out_mode <= 3) || out_mode == TC_OUT_CLAMPED, "rl_gemm_tc_grouped: unknown output mode %d", out_mode);
+  RL_REQUIRE(!tc_out_gated(out_mode) || N % 2 == 0, "rl_gemm_tc_grouped: the gated epilogue needs an even number of weight rows, got %d", N);
+  RL_REQUIRE(ldo >= (tc_out_gated(out_mode) ? N / 2 : N) && err != nullptr && tile_group != nullptr && groups > 0,
              "rl_gemm_tc_grouped: bad output stride, null error word or no groups");
   RL_REQUIRE((bt == 16 || bt == 32 || bt == 64 || bt == 128 || bt == 256) && M % bt == 0,
              "rl_gemm_tc_grouped: the token tile must be 16, 32, 64, 128 or 256 and divide M (%d, %d)", bt, M);
   RL_REQUIRE((long long)groups * N <= 2147483647LL && M / bt <= 65535, "rl_gemm_tc_grouped: too many weight rows or token tiles");
   TcFuse fuse = {};
   fuse.tile_group = tile_group; fuse.group_rows = N;
+  fuse.act_limit = act_limit; fuse.act_alpha = act_alpha;
   fuse.norm_count = 4 * ((N + BLOCK_N_OUT - 1) / BLOCK_N_OUT);
   const int total_kb = (K + BLOCK_K - 1) / BLOCK_K;
   CUtensorMap mw, ma;
@@ -867,8 +886,8 @@ extern "C" int rl_gemm_tc_grouped(const void* A, const void* W, void* out, int o
     case 32: return launch_tc_as<32, false>(mw, ma, nullptr, out, out_mode, M, N, K, ldo, err, 1, total_kb, fuse, stream);
     case 64: return launch_tc_as<64, false>(mw, ma, nullptr, out, out_mode, M, N, K, ldo, err, 1, total_kb, fuse, stream);
     // many tokens an expert: the persistent kernel (an accumulator drains while the next tile's products run)
-    case 128: return launch_tc_persistent<128>(mw, ma, A, lda, nullptr, out, out_mode, M, N, K, ldo, err, stream, tile_group, N);
-    default: return launch_tc_persistent<256>(mw, ma, A, lda, nullptr, out, out_mode, M, N, K, ldo, err, stream, tile_group, N);
+    case 128: return launch_tc_persistent<128>(mw, ma, A, lda, nullptr, out, out_mode, M, N, K, ldo, err, stream, fuse);
+    default: return launch_tc_persistent<256>(mw, ma, A, lda, nullptr, out, out_mode, M, N, K, ldo, err, stream, fuse);
   }
 }
 

@@ -188,7 +188,7 @@ extern "C" int rl_qk_rotate_unit(const void* u, int ldu, void* q_out, int ldq, i
   const dim3 grid(num_tokens, (num_heads + num_kv_heads + HP_WARPS - 1) / HP_WARPS);
   // neighbouring pairs (or no rotation at all) on even sizes and addresses of whole pairs: a pair a load
   const uintptr_t two = dtype == RL_F32 ? 8 : 4;
-  const bool pairs = (interleaved || rotary_dim == 0) && head_dim % 2 == 0 && ldu % 2 == 0 && ldq % 2 == 0 &&
+  const bool pairs = head_dim % 2 == 0 && ldu % 2 == 0 && ldq % 2 == 0 &&
                      (uintptr_t)u % two == 0 && (uintptr_t)q_out % two == 0 && (uintptr_t)k_pool % two == 0 && (uintptr_t)v_pool % two == 0;
   if (pairs && dtype == RL_F32)
     rl_launch_pdl(qk_rotate_unit_pairs_kernel<float>, grid, HP_WARPS * 32, 0, stream, (const float*)u, ldu, (float*)q_out, ldq, positions,
@@ -227,7 +227,7 @@ __device__ __forceinline__ float hp_block_sum(float v, float* s_part) {
 
 // the element i of a rotary part of width rd whose first `rot` dimensions turn: (u, v) -> (u c - v s, v c + u s)
 template <typename T>
-__device__ __forceinline__ float hp_turned(const T* part, int i, int rot, int interleaved, int pos, const float* inv_freq) {
+__device__ __forceinline__ float hp_turned(const T* part, int i, int rot, int interleaved, int pos, const float* inv_freq, float magnitude) {
   const float mine = rl_ld(part + i);
   if (i >= rot) return mine;
   const int half = rot / 2;
@@ -237,7 +237,34 @@ __device__ __forceinline__ float hp_turned(const T* part, int i, int rot, int in
   const float other = rl_ld(part + partner);
   float sn, cs;
   sincosf((float)pos * inv_freq[pair], &sn, &cs);
+  sn *= magnitude;
+  cs *= magnitude;
   return first ? mine * cs - other * sn : mine * cs + other * sn;
+}
+
+// Pair j (of rd / 2) of a part of rd elements, both elements at once: turned among the first `rot`, copied behind them.
+// Accesses are two elements wide except where the pairs are the two halves.
+template <typename T>
+__device__ __forceinline__ void hp_turn_pair(const T* src, T* dst, int j, int rot, int interleaved, int pos, const float* inv_freq,
+                                             float magnitude) {
+  const int half = rot >> 1;
+  if (j >= half) {                       // behind the turned pairs
+    const float2 v = hp_ld2(src + 2 * j);
+    hp_st2(dst + 2 * j, v.x, v.y);
+    return;
+  }
+  float sn, cs;
+  sincosf((float)pos * inv_freq[j], &sn, &cs);
+  sn *= magnitude;
+  cs *= magnitude;
+  if (interleaved) {
+    const float2 v = hp_ld2(src + 2 * j);
+    hp_st2(dst + 2 * j, v.x * cs - v.y * sn, v.y * cs + v.x * sn);
+  } else {
+    const float x = rl_ld(src + j), y = rl_ld(src + j + half);
+    rl_st(dst + j, x * cs - y * sn);
+    rl_st(dst + j + half, y * cs + x * sn);
+  }
 }
 
 template <typename T>
@@ -245,7 +272,7 @@ __global__ void __launch_bounds__(HP_THREADS)
 latent_prepare_kernel(const T* __restrict__ u, int ldu, int q_rank, int kv_rank, int rd, const float* __restrict__ q_w,
                       const float* __restrict__ kv_w, float eps, T* __restrict__ cq, int ldc, const int* __restrict__ positions,
                       const int* __restrict__ slot_of_token, const int* __restrict__ page_table, int max_pages,
-                      const float* __restrict__ inv_freq, int rot, int interleaved, T* __restrict__ k_pool) {
+                      const float* __restrict__ inv_freq, int rot, int interleaved, float magnitude, T* __restrict__ k_pool) {
   __shared__ float s_part[HP_THREADS / 32];
   rl_pdl_trigger();
   rl_pdl_wait();
@@ -273,17 +300,17 @@ latent_prepare_kernel(const T* __restrict__ u, int ldu, int q_rank, int kv_rank,
   const int page = page_table[(size_t)slot * max_pages + pos / RL_PAGE];
   T* dst = k_pool + ((size_t)page * RL_PAGE + pos % RL_PAGE) * (kv_rank + rd);
   for (int i = threadIdx.x; i < kv_rank; i += HP_THREADS) rl_st(dst + i, rl_ld(c + i) * r * kv_w[i]);
-  for (int i = threadIdx.x; i < rd; i += HP_THREADS) rl_st(dst + kv_rank + i, hp_turned(c + kv_rank, i, rot, interleaved, pos, inv_freq));
+  for (int i = threadIdx.x; i < rd; i += HP_THREADS) rl_st(dst + kv_rank + i, hp_turned(c + kv_rank, i, rot, interleaved, pos, inv_freq, magnitude));
 }
 
-// The same with a thread owning neighbouring pairs (all widths, strides and offsets even; rotation of neighbours
-// or none): accesses of twice the width, one sine and cosine a pair.
+// The same with a thread owning pairs (all widths, strides and offsets even): accesses of twice the width, one sine
+// and cosine a pair.
 template <typename T>
 __global__ void __launch_bounds__(HP_THREADS)
 latent_prepare_pairs_kernel(const T* __restrict__ u, int ldu, int q_rank, int kv_rank, int rd, const float* __restrict__ q_w,
                             const float* __restrict__ kv_w, float eps, T* __restrict__ cq, int ldc, const int* __restrict__ positions,
                             const int* __restrict__ slot_of_token, const int* __restrict__ page_table, int max_pages,
-                            const float* __restrict__ inv_freq, int rot, T* __restrict__ k_pool) {
+                            const float* __restrict__ inv_freq, int rot, int interleaved, float magnitude, T* __restrict__ k_pool) {
   __shared__ float s_part[HP_THREADS / 32];
   rl_pdl_trigger();
   rl_pdl_wait();
@@ -317,23 +344,17 @@ latent_prepare_pairs_kernel(const T* __restrict__ u, int ldu, int q_rank, int kv
     const float2 v = hp_ld2(c + i);
     hp_st2(dst + i, v.x * r * kv_w[i], v.y * r * kv_w[i + 1]);
   }
-  for (int i = 2 * threadIdx.x; i < rd; i += 2 * HP_THREADS) {
-    float2 v = hp_ld2(c + kv_rank + i);
-    if (i < rot) {
-      float sn, cs;
-      sincosf((float)pos * inv_freq[i >> 1], &sn, &cs);
-      v = make_float2(v.x * cs - v.y * sn, v.y * cs + v.x * sn);
-    }
-    hp_st2(dst + kv_rank + i, v.x, v.y);
-  }
+  for (int j = threadIdx.x; j < rd / 2; j += HP_THREADS)
+    hp_turn_pair(c + kv_rank, dst + kv_rank, j, rot, interleaved, pos, inv_freq, magnitude);
 }
 
 // u [M, ldu] with columns [0, q_rank) | [q_rank, q_rank + kv_rank) | [.., + rd); q_w float [q_rank], kv_w float [kv_rank];
 // cq [M, ldc]; k_pool [pages, 1, RL_PAGE, kv_rank + rd] (null: nothing is cached).  q_rank 0: no query latent.
+// magnitude: a factor on every cosine and sine.
 extern "C" int rl_latent_prepare(const void* u, int ldu, int dtype, int q_rank, int kv_rank, int rot_dim, const float* q_w,
                                  const float* kv_w, float eps, void* cq, int ldc, const int* positions, const int* slot_of_token,
                                  const int* page_table, int max_pages, const float* inv_freq, int rotary_dim, int interleaved,
-                                 int num_tokens, void* k_pool, cudaStream_t stream) {
+                                 float magnitude, int num_tokens, void* k_pool, cudaStream_t stream) {
   RL_REQUIRE(num_tokens >= 0 && q_rank >= 0 && kv_rank > 0 && rot_dim >= 0, "rl_latent_prepare: bad sizes");
   RL_REQUIRE(rotary_dim >= 0 && rotary_dim <= rot_dim && rotary_dim % 2 == 0, "rl_latent_prepare: rotary width %d must be even and <= %d",
              rotary_dim, rot_dim);
@@ -341,23 +362,24 @@ extern "C" int rl_latent_prepare(const void* u, int ldu, int dtype, int q_rank, 
   RL_REQUIRE(kv_w != nullptr && (q_rank == 0 || (q_w != nullptr && cq != nullptr)), "rl_latent_prepare: a norm weight or the output is missing");
   if (num_tokens == 0) return RL_OK;
   const uintptr_t two = dtype == RL_F32 ? 8 : 4;
-  const bool pairs = (interleaved || rotary_dim == 0) && q_rank % 2 == 0 && kv_rank % 2 == 0 && rot_dim % 2 == 0 && ldu % 2 == 0 &&
+  const bool pairs = q_rank % 2 == 0 && kv_rank % 2 == 0 && rot_dim % 2 == 0 && ldu % 2 == 0 &&
                      ldc % 2 == 0 && (uintptr_t)u % two == 0 && (uintptr_t)cq % two == 0 && (uintptr_t)k_pool % two == 0;
   if (pairs && dtype == RL_F32)
     rl_launch_pdl(latent_prepare_pairs_kernel<float>, num_tokens, HP_THREADS, 0, stream, (const float*)u, ldu, q_rank, kv_rank, rot_dim,
-                  q_w, kv_w, eps, (float*)cq, ldc, positions, slot_of_token, page_table, max_pages, inv_freq, rotary_dim, (float*)k_pool);
+                  q_w, kv_w, eps, (float*)cq, ldc, positions, slot_of_token, page_table, max_pages, inv_freq, rotary_dim,
+                  interleaved, magnitude, (float*)k_pool);
   else if (pairs && dtype == RL_BF16)
     rl_launch_pdl(latent_prepare_pairs_kernel<__nv_bfloat16>, num_tokens, HP_THREADS, 0, stream, (const __nv_bfloat16*)u, ldu, q_rank,
                   kv_rank, rot_dim, q_w, kv_w, eps, (__nv_bfloat16*)cq, ldc, positions, slot_of_token, page_table, max_pages, inv_freq,
-                  rotary_dim, (__nv_bfloat16*)k_pool);
+                  rotary_dim, interleaved, magnitude, (__nv_bfloat16*)k_pool);
   else if (dtype == RL_F32)
     rl_launch_pdl(latent_prepare_kernel<float>, num_tokens, HP_THREADS, 0, stream, (const float*)u, ldu, q_rank, kv_rank, rot_dim, q_w,
-                  kv_w, eps, (float*)cq, ldc, positions, slot_of_token, page_table, max_pages, inv_freq, rotary_dim, interleaved,
+                  kv_w, eps, (float*)cq, ldc, positions, slot_of_token, page_table, max_pages, inv_freq, rotary_dim, interleaved, magnitude,
                   (float*)k_pool);
   else if (dtype == RL_BF16)
     rl_launch_pdl(latent_prepare_kernel<__nv_bfloat16>, num_tokens, HP_THREADS, 0, stream, (const __nv_bfloat16*)u, ldu, q_rank, kv_rank,
                   rot_dim, q_w, kv_w, eps, (__nv_bfloat16*)cq, ldc, positions, slot_of_token, page_table, max_pages, inv_freq,
-                  rotary_dim, interleaved, (__nv_bfloat16*)k_pool);
+                  rotary_dim, interleaved, magnitude, (__nv_bfloat16*)k_pool);
   else
     RL_REQUIRE(false, "rl_latent_prepare: unknown dtype %d", dtype);
   RL_LAUNCH_CHECK("rl_latent_prepare");
@@ -367,7 +389,7 @@ extern "C" int rl_latent_prepare(const void* u, int ldu, int dtype, int q_rank, 
 template <typename T>
 __global__ void __launch_bounds__(HP_THREADS)
 latent_query_kernel(const T* __restrict__ q, int ldq, int H, int hd, int rd, const int* __restrict__ positions,
-                    const float* __restrict__ inv_freq, int rot, int interleaved, T* __restrict__ out, int ldo, int lat) {
+                    const float* __restrict__ inv_freq, int rot, int interleaved, float magnitude, T* __restrict__ out, int ldo, int lat) {
   rl_pdl_trigger();
   rl_pdl_wait();
   const int m = blockIdx.x;
@@ -375,34 +397,29 @@ latent_query_kernel(const T* __restrict__ q, int ldq, int H, int hd, int rd, con
   for (int e = threadIdx.x; e < H * rd; e += HP_THREADS) {
     const int h = e / rd, i = e % rd;
     const T* part = q + (size_t)m * ldq + (size_t)h * (hd + rd) + hd;
-    rl_st(out + (size_t)m * ldo + (size_t)h * (lat + rd) + lat + i, hp_turned(part, i, rot, interleaved, pos, inv_freq));
+    rl_st(out + (size_t)m * ldo + (size_t)h * (lat + rd) + lat + i, hp_turned(part, i, rot, interleaved, pos, inv_freq, magnitude));
   }
 }
 
 template <typename T>
 __global__ void __launch_bounds__(HP_THREADS)
 latent_query_pairs_kernel(const T* __restrict__ q, int ldq, int H, int hd, int rd, const int* __restrict__ positions,
-                          const float* __restrict__ inv_freq, int rot, T* __restrict__ out, int ldo, int lat) {
+                          const float* __restrict__ inv_freq, int rot, int interleaved, float magnitude, T* __restrict__ out, int ldo, int lat) {
   rl_pdl_trigger();
   rl_pdl_wait();
   const int m = blockIdx.x;
   const int pos = positions[m];
   const int half = rd >> 1;
   for (int e = threadIdx.x; e < H * half; e += HP_THREADS) {
-    const int h = e / half, i = 2 * (e % half);
-    float2 v = hp_ld2(q + (size_t)m * ldq + (size_t)h * (hd + rd) + hd + i);
-    if (i < rot) {
-      float sn, cs;
-      sincosf((float)pos * inv_freq[i >> 1], &sn, &cs);
-      v = make_float2(v.x * cs - v.y * sn, v.y * cs + v.x * sn);
-    }
-    hp_st2(out + (size_t)m * ldo + (size_t)h * (lat + rd) + lat + i, v.x, v.y);
+    const int h = e / half, j = e % half;
+    hp_turn_pair(q + (size_t)m * ldq + (size_t)h * (hd + rd) + hd, out + (size_t)m * ldo + (size_t)h * (lat + rd) + lat, j, rot, interleaved,
+                 pos, inv_freq, magnitude);
   }
 }
 
 // q [M, ldq]: H heads of [hd | rd]; out [M, ldo]: H heads of [lat | rd], of which this fills the rd columns.
 extern "C" int rl_latent_query(const void* q, int ldq, int dtype, int num_heads, int head_dim, int rot_dim, const int* positions,
-                               const float* inv_freq, int rotary_dim, int interleaved, void* out, int ldo, int latent_dim,
+                               const float* inv_freq, int rotary_dim, int interleaved, float magnitude, void* out, int ldo, int latent_dim,
                                int num_tokens, cudaStream_t stream) {
   RL_REQUIRE(num_tokens >= 0 && num_heads > 0 && head_dim > 0 && rot_dim >= 0 && latent_dim > 0, "rl_latent_query: bad sizes");
   RL_REQUIRE(rotary_dim >= 0 && rotary_dim <= rot_dim && rotary_dim % 2 == 0, "rl_latent_query: rotary width %d must be even and <= %d",
@@ -410,20 +427,20 @@ extern "C" int rl_latent_query(const void* q, int ldq, int dtype, int num_heads,
   RL_REQUIRE(ldq >= num_heads * (head_dim + rot_dim) && ldo >= num_heads * (latent_dim + rot_dim), "rl_latent_query: row strides too small");
   if (num_tokens == 0 || rot_dim == 0) return RL_OK;
   const uintptr_t two = dtype == RL_F32 ? 8 : 4;
-  const bool pairs = (interleaved || rotary_dim == 0) && head_dim % 2 == 0 && rot_dim % 2 == 0 && latent_dim % 2 == 0 && ldq % 2 == 0 &&
+  const bool pairs = head_dim % 2 == 0 && rot_dim % 2 == 0 && latent_dim % 2 == 0 && ldq % 2 == 0 &&
                      ldo % 2 == 0 && (uintptr_t)q % two == 0 && (uintptr_t)out % two == 0;
   if (pairs && dtype == RL_F32)
     rl_launch_pdl(latent_query_pairs_kernel<float>, num_tokens, HP_THREADS, 0, stream, (const float*)q, ldq, num_heads, head_dim, rot_dim,
-                  positions, inv_freq, rotary_dim, (float*)out, ldo, latent_dim);
+                  positions, inv_freq, rotary_dim, interleaved, magnitude, (float*)out, ldo, latent_dim);
   else if (pairs && dtype == RL_BF16)
     rl_launch_pdl(latent_query_pairs_kernel<__nv_bfloat16>, num_tokens, HP_THREADS, 0, stream, (const __nv_bfloat16*)q, ldq, num_heads,
-                  head_dim, rot_dim, positions, inv_freq, rotary_dim, (__nv_bfloat16*)out, ldo, latent_dim);
+                  head_dim, rot_dim, positions, inv_freq, rotary_dim, interleaved, magnitude, (__nv_bfloat16*)out, ldo, latent_dim);
   else if (dtype == RL_F32)
     rl_launch_pdl(latent_query_kernel<float>, num_tokens, HP_THREADS, 0, stream, (const float*)q, ldq, num_heads, head_dim, rot_dim,
-                  positions, inv_freq, rotary_dim, interleaved, (float*)out, ldo, latent_dim);
+                  positions, inv_freq, rotary_dim, interleaved, magnitude, (float*)out, ldo, latent_dim);
   else if (dtype == RL_BF16)
     rl_launch_pdl(latent_query_kernel<__nv_bfloat16>, num_tokens, HP_THREADS, 0, stream, (const __nv_bfloat16*)q, ldq, num_heads,
-                  head_dim, rot_dim, positions, inv_freq, rotary_dim, interleaved, (__nv_bfloat16*)out, ldo, latent_dim);
+                  head_dim, rot_dim, positions, inv_freq, rotary_dim, interleaved, magnitude, (__nv_bfloat16*)out, ldo, latent_dim);
   else
     RL_REQUIRE(false, "rl_latent_query: unknown dtype %d", dtype);
   RL_LAUNCH_CHECK("rl_latent_query");
@@ -438,7 +455,7 @@ extern "C" int rl_latent_query(const void* q, int ldq, int dtype, int num_heads,
 template <typename T>
 __global__ void __launch_bounds__(256)
 heads_linear_kernel(const T* __restrict__ x, int ldx, int x_head, const T* __restrict__ w, T* __restrict__ out, int ldo,
-                    int out_head, int M, int N, int K) {
+                    int out_head, int M, int N, int K, const T* __restrict__ gate, int ldg) {
   extern __shared__ float hl_x[];          // [HL_TOKENS][K]
   const int a = blockIdx.y, m0 = blockIdx.z * HL_TOKENS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -464,26 +481,33 @@ heads_linear_kernel(const T* __restrict__ x, int ldx, int x_head, const T* __res
     const float v = rl_warp_sum(acc[m]);
     if (lane == m) mine = v;
   }
-  if (lane < HL_TOKENS && m0 + lane < M) rl_st(out + (size_t)(m0 + lane) * ldo + (size_t)a * out_head + n, mine);
+  if (lane < HL_TOKENS && m0 + lane < M) {
+    if (gate) mine *= 1.0f / (1.0f + expf(-rl_ld(gate + (size_t)(m0 + lane) * ldg + (size_t)a * N + n)));
+    rl_st(out + (size_t)(m0 + lane) * ldo + (size_t)a * out_head + n, mine);
+  }
 }
 
 // x: [M, ldx] with head a's K inputs at columns [a * x_head, a * x_head + K); w: [H, N, K] contiguous; out: [M, ldo]
-// with head a's N outputs at columns [a * out_head, a * out_head + N); all of one dtype, sums in 32-bit.
+// with head a's N outputs at columns [a * out_head, a * out_head + N); all of one dtype, sums in 32-bit.  gate (may be
+// null): [M, ldg] with head a's N values at columns [a * N, a * N + N); an output is multiplied by its sigmoid.
 extern "C" int rl_heads_linear(const void* x, int ldx, int x_head, const void* w, void* out, int ldo, int out_head, int dtype,
-                               int M, int H, int N, int K, cudaStream_t stream) {
+                               int M, int H, int N, int K, const void* gate, int ldg, cudaStream_t stream) {
   RL_REQUIRE(M >= 0 && H > 0 && N > 0 && K > 0 && H <= 65535, "rl_heads_linear: bad sizes");
   RL_REQUIRE(ldx >= (H - 1) * x_head + K && ldo >= (H - 1) * out_head + N && x_head >= 0 && out_head >= N,
              "rl_heads_linear: row strides too small for the heads");
+  RL_REQUIRE(gate == nullptr || ldg >= H * N, "rl_heads_linear: the gate's row stride is too small");
   const size_t smem = (size_t)HL_TOKENS * K * sizeof(float);
   RL_REQUIRE(smem <= 48 * 1024, "rl_heads_linear: %d inputs a head exceed the %d this kernel holds", K, 48 * 1024 / (HL_TOKENS * 4));
   if (M == 0) return RL_OK;
   const dim3 grid((N + 7) / 8, H, (M + HL_TOKENS - 1) / HL_TOKENS);
   RL_REQUIRE(grid.z <= 65535, "rl_heads_linear: too many tokens (%d) for this kernel", M);
   if (dtype == RL_F32)
-    heads_linear_kernel<float><<<grid, 256, smem, stream>>>((const float*)x, ldx, x_head, (const float*)w, (float*)out, ldo, out_head, M, N, K);
+    heads_linear_kernel<float><<<grid, 256, smem, stream>>>((const float*)x, ldx, x_head, (const float*)w, (float*)out, ldo, out_head, M, N, K,
+                                                           (const float*)gate, ldg);
   else if (dtype == RL_BF16)
     heads_linear_kernel<__nv_bfloat16><<<grid, 256, smem, stream>>>((const __nv_bfloat16*)x, ldx, x_head, (const __nv_bfloat16*)w,
-                                                                   (__nv_bfloat16*)out, ldo, out_head, M, N, K);
+                                                                   (__nv_bfloat16*)out, ldo, out_head, M, N, K,
+                                                                   (const __nv_bfloat16*)gate, ldg);
   else
     RL_REQUIRE(false, "rl_heads_linear: unknown dtype %d", dtype);
   RL_LAUNCH_CHECK("rl_heads_linear");

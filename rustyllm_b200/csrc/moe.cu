@@ -6,6 +6,9 @@
 //   expert : y_e = Wdown_e (silu(Wgate_e h) * (Wup_e h))
 //   output : residual += sum_c weight_c * y_{e_c}     (choices in the order of falling logits)
 //
+// The gate's activation is an argument: 0 silu(g) * u; 1 g = min(g, limit), u = clamp(u, -limit, limit),
+// g sigmoid(alpha g) (u + 1).
+//
 // Every token is computed by itself, its sums in an order that its own sizes fix, so a token's
 // result does not depend on the batch.  Weights: gate_up [E, 2, F, d] (an expert's gate rows,
 // then its up rows), down [E, d, F].
@@ -182,10 +185,12 @@ extern "C" int rl_moe_route(const void* x, int ldx, const void* router, const fl
 // [2 * groups] are scratch.
 // Variants, each an argument: `softmax_all` - the scores are the softmax of the logits over all experts instead of
 // their sigmoids; `group_top` - a group's score is the sum of its `group_top` largest choice scores (2 above; 1: its
-// largest); `renorm` - the weights are the chosen scores divided by their sum (+ 1e-20).
+// largest); `renorm` - the weights are the chosen scores divided by their sum (+ 1e-20); `weight_scale` - a constant
+// on every weight.
 __device__ __forceinline__ void moe_pick_sigmoid(float* s_score, float* s_choice, float* s_group, const float* __restrict__ correction,
                                                  int E, int top, int groups, int keep, int lane, int* __restrict__ ids,
-                                                 float* __restrict__ weights, int softmax_all = 0, int group_top = 2, int renorm = 0) {
+                                                 float* __restrict__ weights, int softmax_all, int group_top, int renorm,
+                                                 float weight_scale) {
   if (softmax_all) {
     float mx = -INFINITY;
     for (int e = lane; e < E; e += 32) mx = fmaxf(mx, s_score[e]);
@@ -271,7 +276,7 @@ __device__ __forceinline__ void moe_pick_sigmoid(float* s_score, float* s_choice
   }
   if (lane < top) {
     ids[lane] = chosen_id;
-    weights[lane] = chosen_w;
+    weights[lane] = chosen_w * weight_scale;
   }
 }
 
@@ -279,7 +284,7 @@ template <typename T>
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_route_sigmoid_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ wr, const float* __restrict__ correction,
                          int d, int E, int top, int groups, int keep, int* __restrict__ ids, float* __restrict__ weights, int softmax_all,
-                         int group_top, int renorm) {
+                         int group_top, int renorm, float weight_scale) {
   extern __shared__ float s_logit[];     // scores [E], choice scores [E], groups [2 * groups], then the token's input [d]
   const int Ep = (E + 3) & ~3;
   float* s_x = s_logit + 4 * Ep;
@@ -289,13 +294,13 @@ moe_route_sigmoid_kernel(const T* __restrict__ x, int ldx, const T* __restrict__
   if (threadIdx.x >= 32) return;
   const size_t m = blockIdx.x;
   moe_pick_sigmoid(s_logit, s_logit + Ep, s_logit + 2 * Ep, correction, E, top, groups, keep, threadIdx.x, ids + m * top, weights + m * top,
-                   softmax_all, group_top, renorm);
+                   softmax_all, group_top, renorm, weight_scale);
 }
 
 // from logits a matrix product has made: one warp a token
 __global__ void __launch_bounds__(32)
 moe_select_sigmoid_kernel(const float* __restrict__ logits, int E, int top, const float* __restrict__ correction, int groups, int keep,
-                          int* __restrict__ ids, float* __restrict__ weights, int softmax_all, int group_top, int renorm) {
+                          int* __restrict__ ids, float* __restrict__ weights, int softmax_all, int group_top, int renorm, float weight_scale) {
   extern __shared__ float s_logit[];
   const int Ep = (E + 3) & ~3;
   rl_pdl_trigger();
@@ -304,7 +309,7 @@ moe_select_sigmoid_kernel(const float* __restrict__ logits, int E, int top, cons
   for (int e = threadIdx.x; e < E; e += 32) s_logit[e] = logits[m * E + e];
   __syncwarp();
   moe_pick_sigmoid(s_logit, s_logit + Ep, s_logit + 2 * Ep, correction, E, top, groups, keep, threadIdx.x, ids + m * top, weights + m * top,
-                   softmax_all, group_top, renorm);
+                   softmax_all, group_top, renorm, weight_scale);
 }
 
 static int moe_sigmoid_args(const char* who, int num_experts, int top, int groups, int keep) {
@@ -319,25 +324,26 @@ static int moe_sigmoid_args(const char* who, int num_experts, int top, int group
 // rl_moe_select_scored / rl_moe_route_scored: the routers above with the variants as arguments (softmax_all,
 // group_top 1 or 2, renorm; see moe_pick_sigmoid); the *_sigmoid entry points are (0, 2, 0).
 extern "C" int rl_moe_select_scored(const float* logits, int num_tokens, int num_experts, int top, const float* correction, int groups,
-                                    int keep, int softmax_all, int group_top, int renorm, int* ids, float* weights, cudaStream_t stream) {
+                                    int keep, int softmax_all, int group_top, int renorm, float weight_scale, int* ids, float* weights,
+                                    cudaStream_t stream) {
   RL_REQUIRE(num_tokens >= 0 && (group_top == 1 || group_top == 2), "rl_moe_select_scored: bad sizes or group_top %d", group_top);
   if (const int rc = moe_sigmoid_args("rl_moe_select_sigmoid", num_experts, top, groups, keep)) return rc;
   if (num_tokens == 0) return RL_OK;
   const size_t smem = (size_t)4 * ((num_experts + 3) & ~3) * sizeof(float);
   rl_launch_pdl(moe_select_sigmoid_kernel, num_tokens, 32, smem, stream, logits, num_experts, top, correction, groups, keep, ids, weights,
-                softmax_all, group_top, renorm);
+                softmax_all, group_top, renorm, weight_scale);
   RL_LAUNCH_CHECK("rl_moe_select_sigmoid");
   return RL_OK;
 }
 
 extern "C" int rl_moe_select_sigmoid(const float* logits, int num_tokens, int num_experts, int top, const float* correction, int groups,
                                      int keep, int* ids, float* weights, cudaStream_t stream) {
-  return rl_moe_select_scored(logits, num_tokens, num_experts, top, correction, groups, keep, 0, 2, 0, ids, weights, stream);
+  return rl_moe_select_scored(logits, num_tokens, num_experts, top, correction, groups, keep, 0, 2, 0, 1.0f, ids, weights, stream);
 }
 
 extern "C" int rl_moe_route_scored(const void* x, int ldx, const void* router, const float* correction, int dtype, int num_tokens,
                                    int hidden, int num_experts, int top, int groups, int keep, int softmax_all, int group_top, int renorm,
-                                   int* ids, float* weights, cudaStream_t stream) {
+                                   float weight_scale, int* ids, float* weights, cudaStream_t stream) {
   RL_REQUIRE(num_tokens >= 0 && hidden > 0 && (group_top == 1 || group_top == 2), "rl_moe_route_sigmoid: bad sizes M=%d d=%d", num_tokens, hidden);
   if (const int rc = moe_sigmoid_args("rl_moe_route_sigmoid", num_experts, top, groups, keep)) return rc;
   if (num_tokens == 0) return RL_OK;
@@ -345,10 +351,12 @@ extern "C" int rl_moe_route_scored(const void* x, int ldx, const void* router, c
   const size_t smem = (size_t)(4 * ((num_experts + 3) & ~3) + hidden) * sizeof(float);
   if (dtype == RL_F32)
     rl_launch_pdl(moe_route_sigmoid_kernel<float>, num_tokens, MOE_THREADS, smem, stream, (const float*)x, ldx, (const float*)router,
-                  correction, hidden, num_experts, top, groups, keep, ids, weights, softmax_all, group_top, renorm);
+                  correction, hidden, num_experts, top, groups, keep, ids, weights, softmax_all, group_top, renorm,
+                  weight_scale);
   else if (dtype == RL_BF16)
     rl_launch_pdl(moe_route_sigmoid_kernel<__nv_bfloat16>, num_tokens, MOE_THREADS, smem, stream, (const __nv_bfloat16*)x, ldx,
-                  (const __nv_bfloat16*)router, correction, hidden, num_experts, top, groups, keep, ids, weights, softmax_all, group_top, renorm);
+                  (const __nv_bfloat16*)router, correction, hidden, num_experts, top, groups, keep, ids, weights, softmax_all, group_top, renorm,
+                  weight_scale);
   else
     RL_REQUIRE(false, "rl_moe_route_sigmoid: unknown dtype %d", dtype);
   RL_LAUNCH_CHECK("rl_moe_route_sigmoid");
@@ -358,7 +366,7 @@ extern "C" int rl_moe_route_scored(const void* x, int ldx, const void* router, c
 extern "C" int rl_moe_route_sigmoid(const void* x, int ldx, const void* router, const float* correction, int dtype, int num_tokens,
                                     int hidden, int num_experts, int top, int groups, int keep, int* ids, float* weights,
                                     cudaStream_t stream) {
-  return rl_moe_route_scored(x, ldx, router, correction, dtype, num_tokens, hidden, num_experts, top, groups, keep, 0, 2, 0, ids, weights,
+  return rl_moe_route_scored(x, ldx, router, correction, dtype, num_tokens, hidden, num_experts, top, groups, keep, 0, 2, 0, 1.0f, ids, weights,
                              stream);
 }
 
@@ -368,7 +376,7 @@ extern "C" int rl_moe_route_sigmoid(const void* x, int ldx, const void* router, 
 template <typename T>
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_gate_up_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ wgu, const int* __restrict__ ids,
-                   int d, int F, int top, T* __restrict__ h, int interleaved) {
+                   int d, int F, int top, T* __restrict__ h, int interleaved, int act, float limit, float alpha) {
   extern __shared__ float s_x[];          // [d]
   rl_pdl_trigger();
   rl_pdl_wait();
@@ -397,7 +405,15 @@ moe_gate_up_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ wgu, 
   }
   g = rl_warp_sum(g);
   u = rl_warp_sum(u);
-  if (lane == 0) rl_st(h + (size_t)pair * F + r, g / (1.0f + expf(-g)) * u);
+  if (lane == 0) {
+    if (act == 1) {
+      g = fminf(g, limit);
+      u = fminf(fmaxf(u, -limit), limit);
+      rl_st(h + (size_t)pair * F + r, g / (1.0f + expf(-alpha * g)) * (u + 1.0f));
+    } else {
+      rl_st(h + (size_t)pair * F + r, g / (1.0f + expf(-g)) * u);
+    }
+  }
 }
 
 // ------------------------------------------------------------------ down of the chosen experts, weighted, into the residual
@@ -438,7 +454,8 @@ moe_down_kernel(const T* __restrict__ h, const T* __restrict__ wd, const int* __
 // h [M * top, F] scratch in the same dtype; residual [M, d] float, added into.
 extern "C" int rl_moe_experts(const void* x, int ldx, const void* gate_up, const void* down, int dtype, const int* ids,
                               const float* weights, int num_tokens, int hidden, int expert_ff, int num_experts, int top,
-                              int interleaved, void* h, float* residual, cudaStream_t stream) {
+                              int interleaved, int act, float limit, float alpha, void* h, float* residual, cudaStream_t stream) {
+  RL_REQUIRE(act == 0 || act == 1, "rl_moe_experts: unknown activation %d", act);
   RL_REQUIRE(num_tokens >= 0 && hidden > 0 && expert_ff > 0 && num_experts > 0 && top > 0,
              "rl_moe_experts: bad sizes M=%d d=%d F=%d E=%d top=%d", num_tokens, hidden, expert_ff, num_experts, top);
   RL_REQUIRE((long long)num_tokens * top <= 65535LL * 1024, "rl_moe_experts: too many (token, choice) pairs for one launch");
@@ -453,12 +470,12 @@ extern "C" int rl_moe_experts(const void* x, int ldx, const void* gate_up, const
     const size_t smem = (size_t)hidden * sizeof(float);
     if (dtype == RL_F32) {
       rl_launch_pdl(moe_gate_up_kernel<float>, g1, MOE_THREADS, smem, stream, (const float*)x + (size_t)m0 * ldx, ldx, (const float*)gate_up,
-                    ids + p0, hidden, expert_ff, top, (float*)h + (size_t)p0 * expert_ff, interleaved);
+                    ids + p0, hidden, expert_ff, top, (float*)h + (size_t)p0 * expert_ff, interleaved, act, limit, alpha);
       rl_launch_pdl(moe_down_kernel<float>, g2, MOE_THREADS, 0, stream, (const float*)h + (size_t)p0 * expert_ff, (const float*)down,
                     ids + p0, weights + p0, hidden, expert_ff, top, residual + (size_t)m0 * hidden);
     } else if (dtype == RL_BF16) {
       rl_launch_pdl(moe_gate_up_kernel<__nv_bfloat16>, g1, MOE_THREADS, smem, stream, (const __nv_bfloat16*)x + (size_t)m0 * ldx, ldx,
-                    (const __nv_bfloat16*)gate_up, ids + p0, hidden, expert_ff, top, (__nv_bfloat16*)h + (size_t)p0 * expert_ff, interleaved);
+                    (const __nv_bfloat16*)gate_up, ids + p0, hidden, expert_ff, top, (__nv_bfloat16*)h + (size_t)p0 * expert_ff, interleaved, act, limit, alpha);
       rl_launch_pdl(moe_down_kernel<__nv_bfloat16>, g2, MOE_THREADS, 0, stream, (const __nv_bfloat16*)h + (size_t)p0 * expert_ff,
                     (const __nv_bfloat16*)down, ids + p0, weights + p0, hidden, expert_ff, top, residual + (size_t)m0 * hidden);
     } else {

@@ -61,7 +61,7 @@ template <typename T>
 __global__ void __launch_bounds__(CONV_THREADS)
 short_conv_kernel(const T* __restrict__ u, int ldu, const float* __restrict__ w, const float* __restrict__ bias, int act, int C,
                   int taps, const int* __restrict__ slot_of_token, const float* __restrict__ state, long long state_stride,
-                  T* __restrict__ out, int ldo) {
+                  T* __restrict__ out, int ldo, int part, long long out_part) {
   rl_pdl_trigger();
   rl_pdl_wait();
   const int m = blockIdx.x;
@@ -71,7 +71,7 @@ short_conv_kernel(const T* __restrict__ u, int ldu, const float* __restrict__ w,
   const float* st = state + (size_t)slot_of_token[m] * state_stride;
   float acc = conv_at(u, ldu, w, st, C, taps, m, n, c, bias ? bias[c] : 0.f);
   if (act == 1) acc = acc / (1.0f + expf(-acc));
-  rl_st(out + (size_t)m * ldo + c, acc);
+  rl_st(out + (size_t)(c / part) * out_part + (size_t)m * ldo + c % part, acc);
 }
 
 template <typename T>
@@ -190,25 +190,34 @@ qkv_prepare_kernel(const T* __restrict__ u, int ldu, T* __restrict__ q_out, int 
 
 // u [M, ldu] (channels [0, C)), w float [C, taps], bias float [C] or null, act 0 none / 1 silu,
 // state float [slots, state_stride] (this convolution's [taps - 1, C] at the given pointer), out [M, ldo].
-extern "C" int rl_short_conv(const void* u, int ldu, int dtype, const float* w, const float* bias, int act, int channels,
+// rl_short_conv_parts: the output as equal parts of `part` channels, each a matrix [M, ldo] of its own, out_part
+// elements apart (rl_short_conv: one part).
+extern "C" int rl_short_conv_parts(const void* u, int ldu, int dtype, const float* w, const float* bias, int act, int channels,
                              int taps, const int* slot_of_token, const float* state, long long state_stride, void* out, int ldo,
-                             int num_tokens, cudaStream_t stream) {
-  RL_REQUIRE(num_tokens >= 0 && channels > 0, "rl_short_conv: bad sizes");
+                             int part, long long out_part, int num_tokens, cudaStream_t stream) {
+  RL_REQUIRE(num_tokens >= 0 && channels > 0 && part > 0 && channels % part == 0, "rl_short_conv: bad sizes");
   RL_REQUIRE(taps >= 1 && taps <= CONV_MAX_TAPS, "rl_short_conv: %d taps outside [1, %d]", taps, CONV_MAX_TAPS);
-  RL_REQUIRE(ldu >= channels && ldo >= channels, "rl_short_conv: row strides too small");
+  RL_REQUIRE(ldu >= channels && ldo >= part, "rl_short_conv: row strides too small");
   RL_REQUIRE(act == 0 || act == 1, "rl_short_conv: unknown activation %d", act);
   if (num_tokens == 0) return RL_OK;
   const dim3 grid(num_tokens, (channels + CONV_THREADS - 1) / CONV_THREADS);
   if (dtype == RL_F32)
     rl_launch_pdl(short_conv_kernel<float>, grid, CONV_THREADS, 0, stream, (const float*)u, ldu, w, bias, act, channels, taps,
-                  slot_of_token, state, state_stride, (float*)out, ldo);
+                  slot_of_token, state, state_stride, (float*)out, ldo, part, out_part);
   else if (dtype == RL_BF16)
     rl_launch_pdl(short_conv_kernel<__nv_bfloat16>, grid, CONV_THREADS, 0, stream, (const __nv_bfloat16*)u, ldu, w, bias, act,
-                  channels, taps, slot_of_token, state, state_stride, (__nv_bfloat16*)out, ldo);
+                  channels, taps, slot_of_token, state, state_stride, (__nv_bfloat16*)out, ldo, part, out_part);
   else
     RL_REQUIRE(false, "rl_short_conv: unknown dtype %d", dtype);
   RL_LAUNCH_CHECK("rl_short_conv");
   return RL_OK;
+}
+
+extern "C" int rl_short_conv(const void* u, int ldu, int dtype, const float* w, const float* bias, int act, int channels,
+                             int taps, const int* slot_of_token, const float* state, long long state_stride, void* out, int ldo,
+                             int num_tokens, cudaStream_t stream) {
+  return rl_short_conv_parts(u, ldu, dtype, w, bias, act, channels, taps, slot_of_token, state, state_stride, out, ldo, channels, 0,
+                             num_tokens, stream);
 }
 
 // After the step's convolutions have run: the state takes the sequence's last taps - 1 inputs.

@@ -19,6 +19,7 @@ F32, BF16 = 0, 1
 OUT_SAME, OUT_F32, OUT_ADD_F32, OUT_SWIGLU = 0, 1, 2, 3
 OUT_GELU = 5        # the tensor-core product alone: bf16 out = gelu_tanh(product)
 OUT_GEGLU = 6       # the tensor-core product alone: as OUT_SWIGLU with gelu_tanh on the gate
+OUT_CLAMPED = 7     # the tensor-core product alone: as OUT_SWIGLU with the clamped gate (constants: ``act``)
 
 _DT = {torch.float32: F32, torch.bfloat16: BF16}
 
@@ -52,9 +53,9 @@ _SIGNATURES = {
     "rl_channel_decay_scan": [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p,
                               _c_void_p, _c_int, _c_void_p, _c_ll, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "rl_moe_route_scored": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                            _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p],
-    "rl_moe_select_scored": [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p,
-                             _c_void_p],
+                            _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p],
+    "rl_moe_select_scored": [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p,
+                             _c_void_p, _c_void_p],
     "rl_rope_kv_write_mixed": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p,
                                _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int,
                                _c_void_p, _c_void_p],
@@ -78,16 +79,28 @@ _SIGNATURES = {
                                 _c_void_p],
     "rl_attention_shared_key_block_tokens": [_c_int, _c_int, _c_int],
     "rl_attention_shared_key_head_blocks": [_c_int, _c_int, _c_int],
-    "rl_heads_linear": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    "rl_heads_linear": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
+                        _c_int, _c_void_p],
     "rl_embedding_pair": [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll,
                           _c_float, _c_ll, _c_ll, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "rl_gelu_tanh": [_c_void_p, _c_void_p, _c_int, _c_ll, _c_void_p],
     "rl_qk_rotate_unit": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p,
                           _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p],
     "rl_latent_prepare": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_int,
-                          _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
-    "rl_latent_query": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p,
+                          _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p],
+    "rl_latent_query": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_float, _c_void_p,
                         _c_int, _c_int, _c_int, _c_void_p],
+    "rl_streams": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
+                   _c_void_p, _c_void_p, _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p],
+    "rl_gated_recurrence": [_c_void_p, _c_ll, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_int, _c_void_p, _c_int,
+                            _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_ll, _c_int, _c_int, _c_void_p],
+    "rl_gated_recurrence_step": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_int, _c_void_p, _c_int,
+                                 _c_int, _c_void_p, _c_int, _c_void_p, _c_ll, _c_int, _c_int, _c_void_p],
+    "rl_gated_recurrence_step_max_part": [],
+    "rl_short_conv_step": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_ll,
+                           _c_void_p, _c_int, _c_void_p],
+    "rl_short_conv_parts": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_ll,
+                            _c_void_p, _c_int, _c_int, _c_ll, _c_int, _c_void_p],
     "rl_short_conv": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_ll,
                       _c_void_p, _c_int, _c_int, _c_void_p],
     "rl_short_conv_state": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll, _c_void_p],
@@ -114,12 +127,12 @@ _SIGNATURES = {
                      _c_void_p],
     "rl_moe_select": [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p],
     "rl_moe_experts": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
-                       _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p],
+                       _c_int, _c_int, _c_int, _c_float, _c_float, _c_void_p, _c_void_p, _c_void_p],
     "rl_moe_plan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p],
     "rl_moe_gather": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "rl_moe_combine": [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "rl_gemm_tc_grouped": [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
-                           _c_void_p, _c_int, _c_int, _c_void_p],
+                           _c_void_p, _c_int, _c_int, _c_float, _c_float, _c_void_p],
     "rl_repeat_penalty": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p],
     "rl_argmax": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p],
     "rl_sample_temperature": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p],
@@ -166,6 +179,9 @@ _SIGNATURES = {
     "rl_gemm_tc_supported": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int],
     "rl_gemm_tc": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                    _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p],
+    "rl_gemm_tc_act": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                       _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_float, _c_float,
+                       _c_void_p],
     "rl_gemm_tc_splits": [_c_int, _c_int, _c_int],
     "rl_gemm_tc_qkv_rope_supported": [_c_int, _c_int, _c_int, _c_int, _c_int, _c_int],
     "rl_gemm_tc_qkv_rope": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p,
@@ -371,11 +387,13 @@ def moe_select(logits: torch.Tensor, top: int, ids: torch.Tensor, weights: torch
 
 
 def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-                residual: torch.Tensor, interleaved: bool = False) -> None:
+                residual: torch.Tensor, interleaved: bool = False, act=None) -> None:
     """residual[m] += sum_c weights[m, c] * down[e] (silu(gate[e] x[m]) * (up[e] x[m])), e = ids[m, c], on the
     CUDA cores (any sizes, float32 or bfloat16 storage): every (token, choice) pair reads its expert's rows,
     which is what a step of few tokens needs.  gate_up: [E, 2, F, d] (an expert's gate rows, then its up
-    rows) or, ``interleaved``, [E, F, 2, d] (gate_r, up_r in turn); down: [E, d, F]."""
+    rows) or, ``interleaved``, [E, F, 2, d] (gate_r, up_r in turn); down: [E, d, F].  ``act`` (limit, alpha): the clamped
+    gate instead of silu, g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    limit, alpha = act if act is not None else (0.0, 0.0)
     _need(x, "x", contiguous=False); _need(gate_up, "gate_up", x.dtype); _need(down, "down", x.dtype)
     _need(ids, "ids", torch.int32); _need(weights, "weights", torch.float32); _need(residual, "residual", torch.float32)
     M, d = x.shape
@@ -388,8 +406,8 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
     assert ids.shape == (M, top) and weights.shape == (M, top)
     h = torch.empty((M * top, F), dtype=x.dtype, device=x.device)
     _check(library().rl_moe_experts(x.data_ptr(), x.stride(0) if M > 1 else d, gate_up.data_ptr(), down.data_ptr(), _dt(x),
-                                    ids.data_ptr(), weights.data_ptr(), M, d, F, E, top, int(bool(interleaved)), h.data_ptr(),
-                                    residual.data_ptr(), _stream()), "rl_moe_experts")
+                                    ids.data_ptr(), weights.data_ptr(), M, d, F, E, top, int(bool(interleaved)), int(act is not None),
+                                    float(limit), float(alpha), h.data_ptr(), residual.data_ptr(), _stream()), "rl_moe_experts")
     _count(2)
 
 
@@ -408,17 +426,20 @@ def moe_experts_grouped_supported(x: torch.Tensor, gate_up: torch.Tensor, down: 
 
 
 def moe_experts_grouped(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-                        residual: torch.Tensor) -> None:
+                        residual: Optional[torch.Tensor], act=None):
     """The same sum as ``moe_experts`` on the tensor cores, for steps of many tokens: the (token, choice) pairs
     are ordered by expert (every expert's rows padded to whole token tiles), gate and up run as one grouped
     product with the activation in its epilogue, down as a second one, and the choices of a token are added
-    into the residual in their order.  gate_up: [E, F, 2, d] (gate_r, up_r in turn), down: [E, d, F], bf16."""
+    into the residual in their order.  gate_up: [E, F, 2, d] (gate_r, up_r in turn), down: [E, d, F], bf16.  ``act``: see
+    ``moe_experts``.  Without ``residual`` nothing is added: returns (y float32 [rows, d], row int32 [M * top]), the
+    experts' unweighted outputs and where each (token, choice) pair's row lies."""
     _need(x, "x", torch.bfloat16, contiguous=False); _need(gate_up, "gate_up", torch.bfloat16); _need(down, "down", torch.bfloat16)
-    _need(ids, "ids", torch.int32); _need(weights, "weights", torch.float32); _need(residual, "residual", torch.float32)
+    _need(ids, "ids", torch.int32); _need(weights, "weights", torch.float32)
+    limit, alpha = act if act is not None else (0.0, 0.0)
     M, d = x.shape
     E, F, two, d2 = gate_up.shape
     top = ids.shape[1]
-    assert two == 2 and d2 == d and down.shape == (E, d, F) and residual.shape == (M, d)
+    assert two == 2 and d2 == d and down.shape == (E, d, F)
     pairs = M * top
     bt = moe_token_tile(M, top, E)
     rows = (pairs + min(pairs, E) * (bt - 1)) // bt * bt
@@ -432,10 +453,15 @@ def moe_experts_grouped(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tens
     lib, st, err = library(), _stream(), _tc_error_word(dev).data_ptr()
     _check(lib.rl_moe_plan(ids.data_ptr(), pairs, E, bt, tiles, row.data_ptr(), tile_group.data_ptr(), st), "rl_moe_plan")
     _check(lib.rl_moe_gather(x.data_ptr(), x.stride(0) if M > 1 else d, row.data_ptr(), pairs, top, d, xs.data_ptr(), st), "rl_moe_gather")
-    _check(lib.rl_gemm_tc_grouped(xs.data_ptr(), gate_up.data_ptr(), h.data_ptr(), OUT_SWIGLU, rows, 2 * F, d, d, F, err,
-                                  tile_group.data_ptr(), E, bt, st), "rl_gemm_tc_grouped")
+    _check(lib.rl_gemm_tc_grouped(xs.data_ptr(), gate_up.data_ptr(), h.data_ptr(), OUT_SWIGLU if act is None else OUT_CLAMPED, rows,
+                                  2 * F, d, d, F, err, tile_group.data_ptr(), E, bt, float(limit), float(alpha), st), "rl_gemm_tc_grouped")
     _check(lib.rl_gemm_tc_grouped(h.data_ptr(), down.data_ptr(), y.data_ptr(), OUT_F32, rows, d, F, F, d, err,
-                                  tile_group.data_ptr(), E, bt, st), "rl_gemm_tc_grouped")
+                                  tile_group.data_ptr(), E, bt, 0.0, 0.0, st), "rl_gemm_tc_grouped")
+    if residual is None:
+        _count(4)
+        return y, row
+    _need(residual, "residual", torch.float32)
+    assert residual.shape == (M, d)
     _check(lib.rl_moe_combine(y.data_ptr(), row.data_ptr(), weights.data_ptr(), M, top, d, residual.data_ptr(), st), "rl_moe_combine")
     _count(5)
 
@@ -456,8 +482,9 @@ def gemm_tc_row_groups_supported(a: torch.Tensor, w: torch.Tensor) -> bool:
 def gemm_tc_row_groups(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile: int) -> None:
     """Several products of equal shape with inputs and weights of their own as one grouped tensor-core product:
     out[g] = a[g] @ w[g].T for a [G, rows, K], w [G, N, K], out [G, rows, N], all bfloat16 and contiguous, ``rows`` a
-    multiple of ``tile`` (the caller pads; what the padding rows hold does not matter, every row is computed by itself)."""
-    _need(a, "a", torch.bfloat16); _need(w, "w", torch.bfloat16); _need(out, "out", torch.bfloat16)
+    multiple of ``tile`` (the caller pads; what the padding rows hold does not matter, every row is computed by itself).
+    ``out`` may be float32 instead."""
+    _need(a, "a", torch.bfloat16); _need(w, "w", torch.bfloat16); _need(out, "out")
     G, rows, Kd = a.shape
     N = w.shape[1]
     assert w.shape == (G, N, Kd) and out.shape == (G, rows, N) and rows % tile == 0
@@ -466,8 +493,10 @@ def gemm_tc_row_groups(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile
     table = _TILE_GROUPS.get(key)
     if table is None:
         table = _TILE_GROUPS[key] = torch.arange(G * per, dtype=torch.int32, device=a.device).div(per, rounding_mode="floor").to(torch.int32)
-    _check(library().rl_gemm_tc_grouped(a.data_ptr(), w.data_ptr(), out.data_ptr(), OUT_SAME, G * rows, N, Kd, Kd, N,
-                                        _tc_error_word(a.device).data_ptr(), table.data_ptr(), G, tile, _stream()), "rl_gemm_tc_grouped")
+    _check(library().rl_gemm_tc_grouped(a.data_ptr(), w.data_ptr(), out.data_ptr(),
+                                        OUT_F32 if out.dtype == torch.float32 else OUT_SAME, G * rows, N, Kd, Kd, N,
+                                        _tc_error_word(a.device).data_ptr(), table.data_ptr(), G, tile, 0.0, 0.0, _stream()),
+           "rl_gemm_tc_grouped")
     _count()
 
 
@@ -712,19 +741,154 @@ def _state_args(state: torch.Tensor):
 def short_conv(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], silu: bool, slot_of_token: torch.Tensor,
                state: torch.Tensor, out: torch.Tensor) -> None:
     """out[t, c] = act(bias[c] + sum_j weight[c, j] * u[t - taps + 1 + j, c]) along each sequence; inputs of earlier
-    steps come from ``state`` (per slot float [taps - 1, C], written by ``short_conv_state`` afterwards)."""
+    steps come from ``state`` (per slot float [taps - 1, C], written by ``short_conv_state`` afterwards).  ``out``: [M, C],
+    or [parts, >= M, C / parts]: equal parts of the channels as matrices of their own."""
     _need(u, "u", contiguous=False); _need(weight, "weight", torch.float32); _need(out, "out", u.dtype, contiguous=False)
     _need(slot_of_token, "slot_of_token", torch.int32)
-    M, C = out.shape
+    M, C = u.shape
     taps = weight.shape[1]
-    assert weight.shape == (C, taps) and u.shape == (M, C) and u.stride(1) == 1 and out.stride(1) == 1
+    part, out_part, ldo = C, 0, out.stride(0)
+    if out.dim() == 3:
+        part, out_part, ldo = out.shape[2], out.stride(0), out.stride(1)
+        assert out.shape[0] * part == C and out.shape[1] >= M and out.stride(2) == 1
+    else:
+        assert out.shape == (M, C) and out.stride(1) == 1
+    assert weight.shape == (C, taps) and u.stride(1) == 1
     if bias is not None:
         _need(bias, "bias", torch.float32)
         assert bias.numel() == C
     sp, ss = _state_args(state)
     assert state.shape[1] >= 4 * (taps - 1) * C
-    _check(library().rl_short_conv(u.data_ptr(), u.stride(0), _dt(u), weight.data_ptr(), _ptr(bias), int(bool(silu)), C, taps,
-                                   slot_of_token.data_ptr(), sp, ss, out.data_ptr(), out.stride(0), M, _stream()), "rl_short_conv")
+    _check(library().rl_short_conv_parts(u.data_ptr(), u.stride(0), _dt(u), weight.data_ptr(), _ptr(bias), int(bool(silu)), C, taps,
+                                         slot_of_token.data_ptr(), sp, ss, out.data_ptr(), ldo, part, out_part, M, _stream()),
+           "rl_short_conv")
+    _count()
+
+
+def short_conv_step(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], silu: bool, seq_slots: torch.Tensor,
+                    state: torch.Tensor, out: torch.Tensor) -> None:
+    """``short_conv`` and ``short_conv_state`` in one kernel for a step of one token a sequence (row m belongs to slot
+    ``seq_slots[m]``)."""
+    _need(u, "u", contiguous=False); _need(weight, "weight", torch.float32); _need(out, "out", u.dtype, contiguous=False)
+    _need(seq_slots, "seq_slots", torch.int32)
+    M, C = u.shape
+    taps = weight.shape[1]
+    assert weight.shape == (C, taps) and out.shape == (M, C) and u.stride(1) == 1 and out.stride(1) == 1 and seq_slots.numel() == M
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        assert bias.numel() == C
+    sp, ss = _state_args(state)
+    assert state.shape[1] >= 4 * (taps - 1) * C
+    _check(library().rl_short_conv_step(u.data_ptr(), u.stride(0), _dt(u), weight.data_ptr(), _ptr(bias), int(bool(silu)), C, taps,
+                                        seq_slots.data_ptr(), M, sp, ss, out.data_ptr(), out.stride(0), _stream()), "rl_short_conv_step")
+    _count()
+
+
+def gated_recurrence(u: torch.Tensor, z: torch.Tensor, z_bias: torch.Tensor, lam: torch.Tensor, rate: float, y: torch.Tensor,
+                     out: torch.Tensor, state: torch.Tensor, cu_seqlens: torch.Tensor, seq_slots: torch.Tensor, q_lens) -> None:
+    """S_t = a_t S_{t-1} + sqrt(1 - a_t^2) i_t u_t, a_t = exp(-rate r_t softplus(lam)), r and i the sigmoids of the two
+    halves of z + z_bias; out_t = S_t gelu_tanh(y_t).  u: [parts, rows >= M, n]; z float32 [parts, rows, 2 n] (r's sums, then
+    i's); z_bias [parts, 2 n]; lam [W]; y, out [M, W]; the state (float [W] a slot) is read from and left in ``state``."""
+    _need(u, "u"); _need(z, "z", torch.float32); _need(z_bias, "z_bias", torch.float32); _need(lam, "lam", torch.float32)
+    _need(y, "y", u.dtype, contiguous=False); _need(out, "out", u.dtype, contiguous=False)
+    _need(cu_seqlens, "cu_seqlens", torch.int32); _need(seq_slots, "seq_slots", torch.int32)
+    M, W = out.shape
+    parts, rows, n = u.shape
+    assert parts * n == W and rows >= M and z.shape == (parts, rows, 2 * n) and z_bias.numel() == 2 * W and lam.numel() == W
+    assert y.shape == (M, W) and y.stride(1) == 1 and out.stride(1) == 1 and len(q_lens) == seq_slots.numel()
+    sp, ss = _state_args(state)
+    assert state.shape[1] >= 4 * W
+    _check(library().rl_gated_recurrence(u.data_ptr(), rows * n, z.data_ptr(), rows * 2 * n, z_bias.data_ptr(), lam.data_ptr(), float(rate),
+                                         y.data_ptr(), y.stride(0), out.data_ptr(), out.stride(0), _dt(u), cu_seqlens.data_ptr(),
+                                         seq_slots.data_ptr(), seq_slots.numel(), max(q_lens), sp, ss, W, n, _stream()),
+           "rl_gated_recurrence")
+    _count()
+
+
+def gated_recurrence_step_supported(part: int) -> bool:
+    return part <= library().rl_gated_recurrence_step_max_part()
+
+
+def gated_recurrence_step(u: torch.Tensor, w: torch.Tensor, z_bias: torch.Tensor, lam: torch.Tensor, rate: float, y: torch.Tensor,
+                          out: torch.Tensor, state: torch.Tensor, seq_slots: torch.Tensor) -> None:
+    """``gated_recurrence`` for a step of one token a sequence, with the products that make z from u: w [parts, 2 n, n];
+    u, y, out [M, W]."""
+    _need(u, "u", contiguous=False); _need(w, "w", u.dtype); _need(z_bias, "z_bias", torch.float32); _need(lam, "lam", torch.float32)
+    _need(y, "y", u.dtype, contiguous=False); _need(out, "out", u.dtype, contiguous=False); _need(seq_slots, "seq_slots", torch.int32)
+    M, W = out.shape
+    parts, n2, n = w.shape
+    assert n2 == 2 * n and parts * n == W and u.shape == (M, W) and y.shape == (M, W) and z_bias.numel() == 2 * W and lam.numel() == W
+    assert u.stride(1) == 1 and y.stride(1) == 1 and out.stride(1) == 1 and seq_slots.numel() == M
+    sp, ss = _state_args(state)
+    assert state.shape[1] >= 4 * W
+    _check(library().rl_gated_recurrence_step(u.data_ptr(), u.stride(0), w.data_ptr(), z_bias.data_ptr(), lam.data_ptr(), float(rate),
+                                              y.data_ptr(), y.stride(0), out.data_ptr(), out.stride(0), _dt(u), seq_slots.data_ptr(), M,
+                                              sp, ss, W, n, _stream()), "rl_gated_recurrence_step")
+    _count()
+
+
+# ----------------------------------------------------------------------------- a residual of several streams
+def _streams_read_args(X, num, coef, norm_weight, out):
+    S, d = X.shape[1], X.shape[2]
+    if coef is not None:
+        _need(coef, "coef", torch.float32)
+        assert coef.numel() == S
+    if norm_weight is not None:
+        _need(norm_weight, "norm_weight", torch.float32); _need(out, "out")
+        assert norm_weight.numel() == d and out.shape == (num, d)
+    return F32 if out is None else _dt(out)
+
+
+def streams_open(x0: torch.Tensor, X: torch.Tensor, coef: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None,
+                 eps: float = 0.0, out: Optional[torch.Tensor] = None) -> None:
+    """X [M, S, d] = x0 [M, d] in every stream; with ``out``: also ``streams_read`` of the result."""
+    _need(x0, "x0", torch.float32); _need(X, "X", torch.float32)
+    M, S, d = X.shape
+    assert x0.shape == (M, d)
+    odt = _streams_read_args(X, M, coef, norm_weight, out)
+    _check(library().rl_streams(0, X.data_ptr(), x0.data_ptr(), None, 1.0, None, None, 0, None, None, None, _ptr(coef), _ptr(norm_weight),
+                                float(eps), None, M, S, d, _ptr(out), odt, _stream()), "rl_streams")
+    _count()
+
+
+def streams_read(X: torch.Tensor, coef: Optional[torch.Tensor], norm_weight: torch.Tensor, eps: float, out: torch.Tensor,
+                 rows: Optional[torch.Tensor] = None) -> None:
+    """out = rms_norm(sum_s coef[s] X[:, s]) * norm_weight (``coef`` None: the plain sum), at the tokens ``rows`` if given."""
+    _need(X, "X", torch.float32)
+    M, S, d = X.shape
+    num = M if rows is None else rows.numel()
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+    odt = _streams_read_args(X, num, coef, norm_weight, out)
+    _check(library().rl_streams(2, X.data_ptr(), None, None, 1.0, None, None, 0, None, None, None, _ptr(coef), _ptr(norm_weight),
+                                float(eps), _ptr(rows), num, S, d, _ptr(out), odt, _stream()), "rl_streams")
+    _count()
+
+
+def streams_join(X: torch.Tensor, y: torch.Tensor, mix: torch.Tensor, to: torch.Tensor, channel_scale: Optional[torch.Tensor] = None,
+                 y_factor: float = 1.0, row: Optional[torch.Tensor] = None, weights: Optional[torch.Tensor] = None,
+                 coef: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                 out: Optional[torch.Tensor] = None) -> None:
+    """X[:, t] <- sum_s mix[s, t] X[:, s] + to[t] * channel_scale * y, all t from the old X; with ``out``: also
+    ``streams_read`` of the result.  y: float32 [M, d] (times ``y_factor``), or, with ``row`` [M * top] and ``weights``
+    [M, top], experts' rows: y = sum_c weights[m, c] * y[row[m * top + c]]."""
+    _need(X, "X", torch.float32); _need(y, "y", torch.float32); _need(mix, "mix", torch.float32); _need(to, "to", torch.float32)
+    M, S, d = X.shape
+    assert mix.numel() == S * S and to.numel() == S and y.shape[-1] == d
+    top = 0
+    if row is not None:
+        _need(row, "row", torch.int32); _need(weights, "weights", torch.float32)
+        top = weights.shape[1]
+        assert weights.shape == (M, top) and row.numel() == M * top and y_factor == 1.0
+    else:
+        assert y.shape == (M, d)
+    if channel_scale is not None:
+        _need(channel_scale, "channel_scale", torch.float32)
+        assert channel_scale.numel() == d
+    odt = _streams_read_args(X, M, coef, norm_weight, out)
+    _check(library().rl_streams(1, X.data_ptr(), None, y.data_ptr(), float(y_factor), _ptr(row), _ptr(weights), top, _ptr(channel_scale),
+                                mix.data_ptr(), to.data_ptr(), _ptr(coef), _ptr(norm_weight), float(eps), None, M, S, d, _ptr(out), odt,
+                                _stream()), "rl_streams")
     _count()
 
 
@@ -814,10 +978,11 @@ def qk_rotate_unit(u: torch.Tensor, q_out: torch.Tensor, positions: torch.Tensor
 def latent_prepare(u: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, q_weight: Optional[torch.Tensor],
                    kv_weight: torch.Tensor, eps: float, cq: Optional[torch.Tensor], positions: torch.Tensor,
                    slot_of_token: torch.Tensor, page_table: torch.Tensor, inv_freq: torch.Tensor, rotary_dim: int,
-                   interleaved: bool, k_pool: Optional[torch.Tensor]) -> None:
+                   interleaved: bool, k_pool: Optional[torch.Tensor], magnitude: float = 1.0) -> None:
     """u [M, >= q_rank + kv_rank + rot_dim] = [query latent | key/value latent | shared rotary key] as projected:
     cq = rms_norm(query latent) * q_weight; the token's key row [rms_norm(key/value latent) * kv_weight | turned rotary
-    key] goes to its page of ``k_pool`` [pages, 1, PAGE_SIZE, kv_rank + rot_dim]."""
+    key] goes to its page of ``k_pool`` [pages, 1, PAGE_SIZE, kv_rank + rot_dim].  ``magnitude``: a factor on every
+    cosine and sine.  ``q_rank`` 0: no query latent (``q_weight`` and ``cq`` may be ``None``)."""
     _need(u, "u", contiguous=False); _need(positions, "positions", torch.int32); _need(inv_freq, "inv_freq", torch.float32)
     _need(kv_weight, "kv_weight", torch.float32)
     M = u.shape[0]
@@ -836,21 +1001,21 @@ def latent_prepare(u: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, q_w
     _check(library().rl_latent_prepare(u.data_ptr(), ldu, _dt(u), int(q_rank), int(kv_rank), int(rot_dim), _ptr(q_weight),
                                        kv_weight.data_ptr(), float(eps), _ptr(cq) if q_rank else None, ldc, positions.data_ptr(),
                                        _ptr(slot_of_token), _ptr(page_table), max_pages, inv_freq.data_ptr(), int(rotary_dim),
-                                       int(bool(interleaved)), M, _ptr(k_pool), _stream()), "rl_latent_prepare")
+                                       int(bool(interleaved)), float(magnitude), M, _ptr(k_pool), _stream()), "rl_latent_prepare")
     _count()
 
 
 def latent_query(q: torch.Tensor, out: torch.Tensor, num_heads: int, head_dim: int, rot_dim: int, latent_dim: int,
-                 positions: torch.Tensor, inv_freq: torch.Tensor, rotary_dim: int, interleaved: bool) -> None:
+                 positions: torch.Tensor, inv_freq: torch.Tensor, rotary_dim: int, interleaved: bool, magnitude: float = 1.0) -> None:
     """q [M, H * (hd + rd)] (a head: [plain | rotary]); the turned rotary parts go behind the ``latent_dim`` columns of
-    each head of ``out`` [M, H * (latent_dim + rd)]."""
+    each head of ``out`` [M, H * (latent_dim + rd)].  ``magnitude``: a factor on every cosine and sine."""
     _need(q, "q", contiguous=False); _need(out, "out", q.dtype); _need(positions, "positions", torch.int32)
     _need(inv_freq, "inv_freq", torch.float32)
     M = q.shape[0]
     assert q.stride(1) == 1 and q.shape[1] == num_heads * (head_dim + rot_dim) and out.shape == (M, num_heads * (latent_dim + rot_dim))
     ldq = q.stride(0) if M > 1 else q.shape[1]
     _check(library().rl_latent_query(q.data_ptr(), ldq, _dt(q), num_heads, head_dim, rot_dim, positions.data_ptr(),
-                                     inv_freq.data_ptr(), int(rotary_dim), int(bool(interleaved)), out.data_ptr(), out.stride(0),
+                                     inv_freq.data_ptr(), int(rotary_dim), int(bool(interleaved)), float(magnitude), out.data_ptr(), out.stride(0),
                                      latent_dim, M, _stream()), "rl_latent_query")
     _count()
 
@@ -858,17 +1023,24 @@ def latent_query(q: torch.Tensor, out: torch.Tensor, num_heads: int, head_dim: i
 HEADS_LINEAR_MAX_K = 768      # inputs a head that ``heads_linear`` holds in shared memory
 
 
-def heads_linear(x: torch.Tensor, x_head: int, w: torch.Tensor, out: torch.Tensor, out_head: int) -> None:
+def heads_linear(x: torch.Tensor, x_head: int, w: torch.Tensor, out: torch.Tensor, out_head: int,
+                 gate: Optional[torch.Tensor] = None) -> None:
     """A product a head in one launch, for few tokens: out[m, a * out_head + n] = sum_k w[a, n, k] x[m, a * x_head + k].
-    x: [M, >= (H - 1) * x_head + K]; w: [H, N, K]; out: [M, >= (H - 1) * out_head + N]; one dtype, sums in 32-bit."""
+    x: [M, >= (H - 1) * x_head + K]; w: [H, N, K]; out: [M, >= (H - 1) * out_head + N]; one dtype, sums in 32-bit.
+    ``gate`` [M, H * N]: every output is multiplied by the sigmoid of its element."""
     _need(x, "x", contiguous=False); _need(w, "w", x.dtype); _need(out, "out", x.dtype, contiguous=False)
     H, N, Kd = w.shape
     M = x.shape[0]
     assert x.stride(1) == 1 and out.stride(1) == 1 and out.shape[0] == M and Kd <= HEADS_LINEAR_MAX_K
     ldx = x.stride(0) if M > 1 else x.shape[1]
     ldo = out.stride(0) if M > 1 else out.shape[1]
+    ldg = 0
+    if gate is not None:
+        _need(gate, "gate", x.dtype, contiguous=False)
+        assert gate.shape == (M, H * N) and gate.stride(1) == 1
+        ldg = gate.stride(0) if M > 1 else H * N
     _check(library().rl_heads_linear(x.data_ptr(), ldx, int(x_head), w.data_ptr(), out.data_ptr(), ldo, int(out_head), _dt(x),
-                                     M, H, N, Kd, _stream()), "rl_heads_linear")
+                                     M, H, N, Kd, _ptr(gate), ldg, _stream()), "rl_heads_linear")
     _count()
 
 
@@ -1006,10 +1178,11 @@ def moe_select_sigmoid(logits: torch.Tensor, correction: Optional[torch.Tensor],
 
 
 def moe_route_scored(x: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int, keep: int,
-                     ids: torch.Tensor, weights: torch.Tensor, softmax_all: bool, group_top: int, renorm: bool) -> None:
+                     ids: torch.Tensor, weights: torch.Tensor, softmax_all: bool, group_top: int, renorm: bool,
+                     weight_scale: float = 1.0) -> None:
     """``moe_route_sigmoid`` with its variants as arguments: ``softmax_all`` - scores are the softmax of the logits over
     all experts; ``group_top`` - a group's score is the sum of its 1 or 2 largest choice scores; ``renorm`` - the
-    weights are the chosen scores over their sum (+ 1e-20)."""
+    weights are the chosen scores over their sum (+ 1e-20); ``weight_scale`` - a constant on every weight."""
     _need(x, "x", contiguous=False); _need(router, "router", x.dtype); _need(ids, "ids", torch.int32)
     _need(weights, "weights", torch.float32)
     M, d = x.shape
@@ -1020,19 +1193,20 @@ def moe_route_scored(x: torch.Tensor, router: torch.Tensor, correction: Optional
         assert correction.numel() == E
     _check(library().rl_moe_route_scored(x.data_ptr(), x.stride(0) if M > 1 else d, router.data_ptr(), _ptr(correction), _dt(x), M, d,
                                          E, int(top), int(groups), int(keep), int(bool(softmax_all)), int(group_top), int(bool(renorm)),
-                                         ids.data_ptr(), weights.data_ptr(), _stream()), "rl_moe_route_scored")
+                                         float(weight_scale), ids.data_ptr(), weights.data_ptr(), _stream()), "rl_moe_route_scored")
     _count()
 
 
 def moe_select_scored(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int, keep: int,
-                      ids: torch.Tensor, weights: torch.Tensor, softmax_all: bool, group_top: int, renorm: bool) -> None:
+                      ids: torch.Tensor, weights: torch.Tensor, softmax_all: bool, group_top: int, renorm: bool,
+                      weight_scale: float = 1.0) -> None:
     """``moe_route_scored``'s second half alone, from float32 logits [M, E]."""
     _need(logits, "logits", torch.float32); _need(ids, "ids", torch.int32); _need(weights, "weights", torch.float32)
     M, E = logits.shape
     assert ids.shape == (M, top) and weights.shape == (M, top)
     _check(library().rl_moe_select_scored(logits.data_ptr(), M, E, int(top), _ptr(correction), int(groups), int(keep),
-                                          int(bool(softmax_all)), int(group_top), int(bool(renorm)), ids.data_ptr(), weights.data_ptr(),
-                                          _stream()), "rl_moe_select_scored")
+                                          int(bool(softmax_all)), int(group_top), int(bool(renorm)), float(weight_scale), ids.data_ptr(),
+                                          weights.data_ptr(), _stream()), "rl_moe_select_scored")
     _count()
 
 
@@ -1127,11 +1301,12 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, out_mode: int,
             bias: Optional[torch.Tensor] = None, force_splits: int = 0,
             row_sumsq: Optional[torch.Tensor] = None, row_eps: float = 0.0,
             norm_weight: Optional[torch.Tensor] = None, norm_out: Optional[torch.Tensor] = None,
-            norm_sumsq: Optional[torch.Tensor] = None) -> None:
+            norm_sumsq: Optional[torch.Tensor] = None, act=None) -> None:
     """out = a @ w.T (+ bias) on the tensor cores (tcgen05).  a: [M, K] bf16, w: [N, K] bf16;
     out: bf16 (OUT_SAME) or float32 (OUT_F32 store, OUT_ADD_F32 add), or, with OUT_SWIGLU,
     bf16 [M, N/2] = silu(even columns) * odd columns of the product, or, with OUT_GELU, bf16 [M, N] = the tanh form
-    of gelu of the product, computed in 32-bit from the accumulator.  force_splits: 0 = the
+    of gelu of the product, computed in 32-bit from the accumulator; OUT_CLAMPED: as OUT_SWIGLU with the clamped gate of
+    ``moe_experts``, ``act`` = (limit, alpha).  force_splits: 0 = the
     kernel's own choice of K parts; 1 to 8 = as given.
 
     An RMSNorm around the product can ride along.  ``row_sumsq`` [M, pieces] float32 with
@@ -1143,7 +1318,9 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, out_mode: int,
     M, K = a.shape
     N = w.shape[0]
     assert w.shape[1] == K and out.stride(1) == 1
-    if out_mode in (OUT_SWIGLU, OUT_GEGLU):      # rows of w are (gate_0, up_0, gate_1, ...): out = act(gate) * up, [M, N/2]
+    assert (act is not None) == (out_mode == OUT_CLAMPED)
+    limit, alpha = act if act is not None else (0.0, 0.0)
+    if out_mode in (OUT_SWIGLU, OUT_GEGLU, OUT_CLAMPED):      # rows of w are (gate_0, up_0, gate_1, ...): out = act(gate) * up, [M, N/2]
         assert N % 2 == 0 and out.shape == (M, N // 2) and out.dtype == torch.bfloat16
     else:
         assert out.shape == (M, N)
@@ -1163,10 +1340,11 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, out_mode: int,
         assert norm_sumsq.shape == (M, norm_pieces(N))
     lda = a.stride(0) if M > 1 else K
     ldo = out.stride(0) if M > 1 else out.shape[1]
-    _check(library().rl_gemm_tc(a.data_ptr(), w.data_ptr(), _ptr(bias), out.data_ptr(), out_mode, M, N, K, lda, ldo,
-                                _tc_error_word(a.device).data_ptr(), int(force_splits),
-                                _ptr(row_sumsq), pieces, float(row_eps),
-                                _ptr(norm_weight), _ptr(norm_out), N, _ptr(norm_sumsq), _stream()), "rl_gemm_tc")
+    _check(library().rl_gemm_tc_act(a.data_ptr(), w.data_ptr(), _ptr(bias), out.data_ptr(), out_mode, M, N, K, lda, ldo,
+                                    _tc_error_word(a.device).data_ptr(), int(force_splits),
+                                    _ptr(row_sumsq), pieces, float(row_eps),
+                                    _ptr(norm_weight), _ptr(norm_out), N, _ptr(norm_sumsq), float(limit), float(alpha), _stream()),
+           "rl_gemm_tc")
     _count()
 
 

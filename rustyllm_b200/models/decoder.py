@@ -17,6 +17,7 @@ from ..config.spec import ModelSpec, ParamSpec
 from ..parts import Runtime
 from ..parts.base import Part
 from ..parts.registry import _REGISTRIES, build_part
+from ..parts.streams import StreamRead, open_streams, read_streams
 
 
 @dataclass
@@ -52,7 +53,12 @@ class DecoderModel:
                 raise KeyError(f"no block of kind {ls.block.kind!r} is registered")
             self.blocks.append(block_cls(runtime=runtime, mixer=mixer, mixer_norm=mixer_norm,
                                          feed_forward=ff, feed_forward_norm=ff_norm, **ls.block.params))
+            if getattr(self.blocks[-1], "streams", 0) != spec.streams:
+                raise ValueError(f"a block of kind {ls.block.kind!r} with {getattr(self.blocks[-1], 'streams', 0)} streams in a model "
+                                 f"with {spec.streams} (0: a plain residual)")
         self.final_norm = build_part("norm", spec.final_norm, runtime)
+        if spec.streams and not hasattr(self.final_norm, "eps"):
+            raise ValueError("a residual of several streams ends in an RMS norm (a weight and an eps)")
         self.head = build_part("head", spec.head, runtime)
         # additions to the residual stream between layers, by the place of the run they stand before
         self.inject_parts = [build_part("inject", ps, runtime) for ps in spec.inject_parts]
@@ -149,7 +155,8 @@ class DecoderModel:
         return made[1]
 
     def forward(self, step, cache: SequenceCache) -> torch.Tensor:
-        """All tokens of the step through all scheduled layers: float32 [M, d]."""
+        """All tokens of the step through all scheduled layers: float32 [M, d] ([M, streams, d] in a model whose
+        residual has several)."""
         nat = self.native_for(cache)
         if nat is not None:
             return nat.forward(step)
@@ -163,6 +170,9 @@ class DecoderModel:
             embedded.copy_(x)
         schedule = self.spec.schedule
         pending = None      # the next block's first norm, started by the block in front of it
+        if self.spec.streams:
+            x, pending = open_streams(x, self.spec.streams, self.runtime.compute_dtype,
+                                      self.blocks[schedule[0]].first_norm_request(x.shape[0]))
         for pos, li in enumerate(schedule):
             for part, args in self.injections.get(pos, ()):
                 part.forward(x, embedded, step, **args)
@@ -194,5 +204,8 @@ class DecoderModel:
         made = getattr(self, "_native", None)
         if self.use_native and made is not None and made[1] is not None:
             return made[1].logits(x, rows)
-        xn = self.final_norm.forward(x, self.runtime.compute_dtype, rows)
+        if self.spec.streams:
+            xn = read_streams(x, StreamRead(None, self.final_norm.weight, self.final_norm.eps), self.runtime.compute_dtype, rows)
+        else:
+            xn = self.final_norm.forward(x, self.runtime.compute_dtype, rows)
         return self.head.forward(xn)

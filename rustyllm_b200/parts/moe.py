@@ -6,6 +6,8 @@ has one, runs for every token and is added.
     C = the ``top`` experts of largest z; w_c = softmax over z restricted to C
     x += sum_{c in C} w_c * Wdown_c (silu(Wgate_c xn) * (Wup_c xn))  [+ shared(xn)]
 
+Other scores, choices, weights and gates that designs use are constructor parameters (see there).
+
 The experts' matrices are stacked: gate and up as [E, 2, F, d] (in a bfloat16 run [E, F, 2, d]: a gate row
 and its up row in turn, as the tensor-core product's SwiGLU epilogue wants them), down as [E, d, F], so one
 kernel indexes any expert.  A bfloat16 step orders its (token, choice) pairs by expert and runs two grouped
@@ -15,6 +17,7 @@ CUDA cores.  The shared expert is an ordinary gated feed-forward part of its own
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Dict, Optional
 
 import torch
@@ -26,11 +29,21 @@ from .linear import OUT_F32, linear
 from .registry import build_part, register_feed_forward
 
 
+@dataclass
+class ExpertRows:
+    """The chosen experts' outputs before they are weighed and summed: token m's choice c is row ``row[m * top + c]`` of
+    ``rows`` and counts ``weights[m, c]``.  For whoever sums them on the way into the residual."""
+    rows: torch.Tensor            # float32 [*, d]
+    row: torch.Tensor             # int32 [M * top]
+    weights: torch.Tensor         # float32 [M, top]
+
+
 @register_feed_forward("moe_mlp")
 class MoEMLP(FeedForward):
     def __init__(self, runtime: Runtime, hidden_size: int, expert_size: int, num_experts: int, top: int,
                  names: Dict[str, str], router_bias: bool = True, shared: Optional[PartSpec] = None,
-                 scoring: str = "softmax", groups: int = 1, keep_groups: int = 1):
+                 scoring: str = "softmax", groups: int = 1, keep_groups: int = 1, weight_scale: float = 1.0,
+                 activation: str = "silu", limit: Optional[float] = None, alpha: Optional[float] = None):
         """``names``: "router" (the router's matrix; its bias is that name + ``names["bias_suffix"]``),
         "expert" (a format string with ``{e}`` for the expert's number, giving the prefix of its
         "gate", "up" and "down" tensors), "suffix" (what follows a projection's name)."""
@@ -46,6 +59,16 @@ class MoEMLP(FeedForward):
         # "sigmoid": scores s = sigmoid(z); experts are chosen by s + correction (``names["correction"]``, a value an
         # expert) among the ``keep_groups`` best of ``groups`` equal groups of neighbours (a group's score: its two
         # largest choice scores); the weights are the chosen experts' s, not renormalised
+        # ``weight_scale``: a constant on every weight (scores other than "softmax").  ``activation`` "clamped_sigmoid":
+        # an expert is Wdown (g sigmoid(alpha g) (u + 1)) with g = min(Wgate x, limit), u = clamp(Wup x, -limit, limit)
+        if activation not in ("silu", "clamped_sigmoid"):
+            raise ValueError(f"activation {activation!r} is not known; known: 'silu', 'clamped_sigmoid'")
+        if activation == "clamped_sigmoid" and (limit is None or alpha is None or not limit > 0):
+            raise ValueError("activation 'clamped_sigmoid' needs limit > 0 and alpha")
+        if weight_scale != 1.0 and scoring == "softmax":
+            raise ValueError("a constant on the weights exists with sigmoid and softmax_all scores only")
+        self.weight_scale = float(weight_scale)
+        self.act = (float(limit), float(alpha)) if activation == "clamped_sigmoid" else None
         self.scoring, self.groups, self.keep_groups = scoring, int(groups), int(keep_groups)
         if scoring in ("sigmoid", "softmax_all"):
             if router_bias:
@@ -108,7 +131,23 @@ class MoEMLP(FeedForward):
     # False: every step on the per-pair kernels (for measurements and tests)
     use_grouped = True
 
-    def forward(self, xn: torch.Tensor, residual: torch.Tensor, step) -> None:
+    offers_rows = True       # ``forward_out(..., rows_ok=True)`` may return ``ExpertRows`` as its term
+
+    def forward_out(self, xn: torch.Tensor, step, rows_ok: bool = False):
+        """The output as a float32 [M, d] term of its own, or (``rows_ok``, where the grouped products made them and no
+        shared expert is added) as the experts' rows."""
+        if rows_ok and self.shared is None and self.interleaved:
+            wgu, wd = self.wgu.view(self.E, self.F, 2, self.d), self.wdown.view(self.E, self.d, self.F)
+            if self.use_grouped and K.moe_experts_grouped_supported(xn, wgu, wd):
+                ids, weights = self.route(xn)
+                rows, row = K.moe_experts_grouped(xn, wgu, wd, ids, weights, None, act=self.act)
+                return [(ExpertRows(rows, row, weights), 1.0)]
+        y = torch.zeros((xn.shape[0], self.d), dtype=torch.float32, device=xn.device)
+        self.forward(xn, y, step)
+        return [(y, 1.0)]
+
+    def route(self, xn: torch.Tensor):
+        """The chosen experts and their weights: (int32 [M, top], float32 [M, top])."""
         M = xn.shape[0]
         ids = torch.empty((M, self.top), dtype=torch.int32, device=xn.device)
         weights = torch.empty((M, self.top), dtype=torch.float32, device=xn.device)
@@ -117,7 +156,7 @@ class MoEMLP(FeedForward):
             raise K.KernelError(f"the router's matrix is {router.dtype} in a {xn.dtype} run")
         if self.scoring in ("sigmoid", "softmax_all"):
             variant = dict(softmax_all=self.scoring == "softmax_all", group_top=1 if self.scoring == "softmax_all" else 2,
-                           renorm=self.scoring == "softmax_all")
+                           renorm=self.scoring == "softmax_all", weight_scale=self.weight_scale)
             if M >= self.ROUTER_PRODUCT_FROM:
                 logits = torch.empty((M, self.E), dtype=torch.float32, device=xn.device)
                 linear(xn, router, logits, OUT_F32)
@@ -131,15 +170,19 @@ class MoEMLP(FeedForward):
             K.moe_select(logits, self.top, ids, weights)
         else:
             K.moe_route(xn, router, self.router_b, self.top, ids, weights)
+        return ids, weights
+
+    def forward(self, xn: torch.Tensor, residual: torch.Tensor, step) -> None:
+        ids, weights = self.route(xn)
         wd = self.wdown.view(self.E, self.d, self.F)
         if self.interleaved:
             wgu = self.wgu.view(self.E, self.F, 2, self.d)
             if self.use_grouped and K.moe_experts_grouped_supported(xn, wgu, wd):
-                K.moe_experts_grouped(xn, wgu, wd, ids, weights, residual)
+                K.moe_experts_grouped(xn, wgu, wd, ids, weights, residual, act=self.act)
             else:
-                K.moe_experts(xn, wgu, wd, ids, weights, residual, interleaved=True)
+                K.moe_experts(xn, wgu, wd, ids, weights, residual, interleaved=True, act=self.act)
         else:
-            K.moe_experts(xn, self.wgu.view(self.E, 2, self.F, self.d), wd, ids, weights, residual)
+            K.moe_experts(xn, self.wgu.view(self.E, 2, self.F, self.d), wd, ids, weights, residual, act=self.act)
         if self.shared_gated and self.shared is not None:
             (y, _), = self.shared.forward_out(xn, step)
             K.row_gate_add(residual, y, xn, self.shared_gate)

@@ -1,6 +1,6 @@
-"""Mixers that carry a matrix state per head from token to token instead of caching keys and values.
+"""Mixers that carry a state from token to token instead of caching keys and values.
 
-Both are the same recurrence, S_t = a_t S_{t-1} + b_t k_t v_t^T with the output o_t = S_t^T q_t (csrc/linear_scan.cu),
+The first two are the same recurrence, S_t = a_t S_{t-1} + b_t k_t v_t^T with the output o_t = S_t^T q_t (csrc/linear_scan.cu),
 with different decays and different parts around it:
 
 ``decay_linear_attention``
@@ -248,6 +248,98 @@ class ShiftedDecayRecurrence(_StateMixer):
         on = torch.empty((M, inner), dtype=dt, device=dev)
         K.gated_norm(o, proj[3], self.norm_w, self.eps, on, groups=H, gate_act="silu", gate_first=False)
         linear(on, self.wo, residual, _out_mode)
+
+
+@register_mixer("gated_linear_recurrence")
+class GatedLinearRecurrence(_StateMixer):
+    """A linear recurrence of one state a channel beside a gelu branch, both ``width`` wide:
+
+        y = gelu_tanh(W_y h + b_y);   u = causal filter over time of (W_x h + b_x), a filter and a bias a channel
+        in ``blocks`` equal parts of the channels:   r = sigmoid(R_a u + b),  i = sigmoid(R_i u + b)
+        log a = -decay_rate * r * softplus(lam);   S_t = a S_{t-1} + sqrt(1 - a^2) i u;   out = W_o (S * y)
+
+    (De et al., "Griffin: Mixing Gated Linear Recurrences with Local Attention for Efficient Language Models".)  The
+    per-sequence state is the filter's last taps - 1 inputs and S, float32, zero for a fresh sequence.  The products'
+    outputs and the filter's take the compute dtype; the gates (from their products' 32-bit sums on), the decay, the
+    input's factor, the state and the product S * y are 32-bit.
+
+    A step of one token a sequence is a product, the filter with the shift of its kept inputs, one kernel for gates,
+    recurrence and gelu branch, and W_o; a step with more runs the gates as one grouped tensor-core product and the
+    recurrence over spans of tokens (csrc/gated_recurrence.cu)."""
+
+    def __init__(self, runtime: Runtime, hidden_size: int, width: int, blocks: int, conv_taps: int, names: Dict[str, str],
+                 decay_rate: float = 8.0):
+        """``names``: "y", "x", "o" (matrices; the first two with biases, + ``names["bias_suffix"]``), "conv" (filters
+        [width, taps], bias likewise), "ra", "ri" (the gates' matrices [blocks, n, n], bias likewise), "lam", "suffix"."""
+        if width <= 0 or blocks <= 0 or width % blocks:
+            raise ValueError(f"{blocks} blocks do not divide a width of {width}")
+        if not (1 <= conv_taps <= 8):
+            raise ValueError(f"conv_taps {conv_taps} outside [1, 8]")
+        self.runtime = runtime
+        self.d, self.W, self.blocks, self.n, self.taps = hidden_size, width, blocks, width // blocks, int(conv_taps)
+        self.rate = float(decay_rate)
+        self.names = names
+        self._conv_bytes = _aligned(4 * (self.taps - 1) * width)
+        self.w_in = self.b_in = self.conv_w = self.conv_b = self.w_gates = self.b_gates = self.lam = self.wo = None
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        d, W, b, n, names = self.d, self.W, self.blocks, self.n, self.names
+        sfx, bsfx = names.get("suffix", ".weight"), names.get("bias_suffix", ".bias")
+
+        def bias(keys, shape):
+            return ParamSpec(tuple(ParamSource(names[k] + bsfx, shape) for k in keys), role="vector", init="zeros")
+        return {
+            "w_in": ParamSpec((ParamSource(names["y"] + sfx, (W, d)), ParamSource(names["x"] + sfx, (W, d)))),
+            "b_in": bias(("y", "x"), (W,)),
+            "conv_w": ParamSpec((ParamSource(names["conv"], (W, self.taps)),), role="vector"),
+            "conv_b": bias(("conv",), (W,)),
+            "w_gates": ParamSpec((ParamSource(names["ra"] + sfx, (b, n, n)), ParamSource(names["ri"] + sfx, (b, n, n)))),
+            "b_gates": bias(("ra", "ri"), (b, n)),
+            "lam": ParamSpec((ParamSource(names["lam"], (W,)),), role="vector", init="normal"),
+            "wo": ParamSpec((ParamSource(names["o"] + sfx, (d, W)),)),
+        }
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        # both gates of a part behind one another: [2, blocks, ...] -> [blocks, 2, ...], so one product serves a part
+        b, n = self.blocks, self.n
+        tensors = dict(tensors)
+        if "w_gates" in tensors:
+            tensors["w_gates"] = tensors["w_gates"].view(2, b, n, n).transpose(0, 1).contiguous().view(b, 2 * n, n)
+        if "b_gates" in tensors:
+            tensors["b_gates"] = tensors["b_gates"].view(2, b, n).transpose(0, 1).contiguous().view(b, 2 * n)
+        super().bind(tensors)
+
+    def state_need(self) -> StateNeed:
+        return StateNeed(self._conv_bytes + 4 * self.W)
+
+    def forward(self, xn, residual: torch.Tensor, step, cache, _out_mode=OUT_ADD_F32):
+        W, b, n = self.W, self.blocks, self.n
+        M, dt, dev = xn.shape[0], xn.dtype, xn.device
+        state = self._state(cache)
+        conv_state, rec_state = state[:, :self._conv_bytes], state[:, self._conv_bytes:]
+        proj = torch.empty((M, 2 * W), dtype=dt, device=dev)
+        linear(xn, self.w_in, proj, OUT_SAME, self.b_in)
+        y, x = proj[:, :W], proj[:, W:]
+        o = torch.empty((M, W), dtype=dt, device=dev)
+        if step.is_decode and self.w_gates.dtype == dt and K.gated_recurrence_step_supported(n):
+            u = torch.empty((M, W), dtype=dt, device=dev)
+            K.short_conv_step(x, self.conv_w, self.conv_b, False, step.seq_slots, conv_state, u)
+            K.gated_recurrence_step(u, self.w_gates, self.b_gates, self.lam, self.rate, y, o, rec_state, step.seq_slots)
+        else:
+            grouped = dt == torch.bfloat16 and self.w_gates.dtype == dt and n % 8 == 0
+            tile = K.gemm_tc_row_groups_tile(M) if grouped else 1
+            rows = -(-M // tile) * tile       # a part's rows padded to whole tiles; the padding's results are not read
+            u = torch.empty((b, rows, n), dtype=dt, device=dev)
+            K.short_conv(x, self.conv_w, self.conv_b, False, step.slot_of_token, conv_state, u)
+            K.short_conv_state(x, self.taps, step.cu_seqlens, step.seq_slots, conv_state)
+            z = torch.empty((b, rows, 2 * n), dtype=torch.float32, device=dev)
+            if grouped:
+                K.gemm_tc_row_groups(u, self.w_gates, z, tile)
+            else:
+                for i in range(b):
+                    linear(u[i], self.w_gates[i], z[i], OUT_F32)
+            K.gated_recurrence(u, z, self.b_gates, self.lam, self.rate, y, o, rec_state, step.cu_seqlens, step.seq_slots, step.q_lens)
+        linear(o, self.wo, residual, _out_mode)
 
 
 @register_mixer("parallel_mixers")
