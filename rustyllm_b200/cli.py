@@ -281,7 +281,11 @@ def run_kernel_benchmark(runner, runs: int, as_json: bool, layer_index: int = 0)
     xn = torch.empty(1, d, device=dev, dtype=dt)
     rows = []
     from .parts.norm import LayerNorm
-    if isinstance(blk.mixer_norm, LayerNorm):
+    if getattr(blk, "streams", 0):        # a residual of several streams: a sublayer's output in, the next one's normed input out
+        X = torch.randn(1, blk.streams, d, device=dev)
+        rows.append(("streams.join_norm", timed(lambda: blk._join(X, [(x, 1.0)], 1, blk.first_norm_request(1))),
+                     (2 * blk.streams + 1) * d * 4 + d * esz))
+    elif isinstance(blk.mixer_norm, LayerNorm):
         rows.append(("attn_norm.layer", timed(lambda: K.layer_norm(x, blk.mixer_norm.weight, xn, blk.mixer_norm.eps)), d * 4))
     else:
         rows.append(("attn_norm.rms", timed(lambda: K.rmsnorm(x, blk.mixer_norm.weight, xn, blk.mixer_norm.eps)), d * 4))
@@ -329,16 +333,7 @@ def run_kernel_benchmark(runner, runs: int, as_json: bool, layer_index: int = 0)
         rows.append(("ffn_up_gelu_down", timed(lambda: ff.forward(xf, x, None)), (ff.wup.numel() + ff.wdown.numel()) * ff.wup.element_size()))
     elif isinstance(ff, MoEMLP):          # router and the chosen experts of one token; the shared expert like a dense one
         xe = xn.to(ff.router.dtype)
-        ids = torch.empty((1, ff.top), dtype=torch.int32, device=dev)
-        wts = torch.empty((1, ff.top), dtype=torch.float32, device=dev)
-        if getattr(ff, "scoring", "softmax") == "softmax_all":
-            rows.append(("ffn_router", timed(lambda: K.moe_route_scored(xe, ff.router, None, ff.top, ff.groups, ff.keep_groups, ids, wts,
-                                                                        softmax_all=True, group_top=1, renorm=True)), ff.router.numel() * esz))
-        elif getattr(ff, "scoring", "softmax") == "sigmoid":
-            rows.append(("ffn_router", timed(lambda: K.moe_route_sigmoid(xe, ff.router, ff.correction, ff.top, ff.groups, ff.keep_groups, ids, wts)),
-                         ff.router.numel() * esz))
-        else:
-            rows.append(("ffn_router", timed(lambda: K.moe_route(xe, ff.router, ff.router_b, ff.top, ids, wts)), ff.router.numel() * esz))
+        rows.append(("ffn_router", timed(lambda: ff.route(xe)), ff.router.numel() * esz))
         shared, ff.shared = ff.shared, None
         try:
             rows.append(("ffn_experts.chosen", timed(lambda: ff.forward(xe, x, None)), ff.router.numel() * esz + ff.top * 3 * ff.F * ff.d * esz))

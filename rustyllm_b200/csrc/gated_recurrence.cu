@@ -5,13 +5,15 @@
 //   log a = -rate * r * softplus(lam);   S_t = exp(log a) S_{t-1} + sqrt(1 - exp(2 log a)) * i * u_t
 //   out_t = S_t * gelu_tanh(y_t)                         (y: the branch beside the recurrence, as projected)
 //
-// The state starts at zero and lives per slot as float [width].  Everything but the stored u, y and out is 32-bit;
-// 1 - exp(2 log a) is formed by expm1, so it keeps its digits where the decay is close to 1.
+// The state starts at zero and lives per slot as float [width].  Everything but the stored u, y and out is 32-bit.
+// Where the decay is close to 1 (a memory of hundreds of tokens and more) exp(log a) has lost the digits that matter:
+// rounded to float it is off by the same amount token after token.  So a step is held as h = exp(log a) - 1 (expm1):
+// S + (h S + b), with 1 - a^2 = -h (2 + h), and a span of steps as expm1 of the sum of their logarithms.
 //
 // rl_gated_recurrence        prompts and portions: the gates' products zr, zi are given (a matrix product a part of
 //                            the channels).  A block owns GR_CH channels of one sequence and walks its tokens in
 //                            spans of TC * GR_STEPS: a thread takes GR_STEPS consecutive tokens of one channel,
-//                            reduces them to one step S -> A S + B, the threads' steps are composed in order
+//                            reduces them to one step of the same form, the threads' steps are composed in order
 //                            through shared memory, and each replays its tokens from its own start.
 // rl_gated_recurrence_step   one token a sequence: the gates' products, the recurrence and the output in one kernel.
 //                            A warp owns a channel (its row of either matrix) for 16 tokens whose inputs wait in
@@ -31,11 +33,16 @@ __device__ __forceinline__ float gr_softplus(float z) { return fmaxf(z, 0.f) + l
 __device__ __forceinline__ float gr_gelu(float z) {
   return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
-// the token's step of the recurrence: S -> a S + b
-__device__ __forceinline__ float2 gr_step(float u, float zr, float zi, float rate_sp) {
-  const float log_a = -rate_sp * gr_sigmoid(zr);
-  return make_float2(expf(log_a), sqrtf(-expm1f(2.0f * log_a)) * gr_sigmoid(zi) * u);
+// the token's step of the recurrence: S -> S + (h S + b); log a
+struct GrStep { float log_a, h, b; };
+__device__ __forceinline__ GrStep gr_step(float u, float zr, float zi, float rate_sp) {
+  GrStep s;
+  s.log_a = -rate_sp * gr_sigmoid(zr);
+  s.h = expm1f(s.log_a);
+  s.b = sqrtf(-s.h * (2.0f + s.h)) * gr_sigmoid(zi) * u;
+  return s;
 }
+__device__ __forceinline__ float gr_advance(float S, float h, float b) { return S + fmaf(h, S, b); }
 
 // u: channel c of token m at u[(c / part) * u_part + m * part + c % part]; z: float, its two sums at
 // z[(c / part) * z_part + m * 2 part + c % part] (decay gate) and + part (input gate).
@@ -45,7 +52,7 @@ gated_recurrence_kernel(const T* __restrict__ u, long long u_part, const float* 
                         const float* __restrict__ z_bias, const float* __restrict__ lam, float rate, const T* __restrict__ y, int ldy,
                         T* __restrict__ out, int ldo, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slots,
                         float* __restrict__ state, long long state_stride, int W, int part) {
-  __shared__ float s_a[TC][GR_CH], s_b[TC][GR_CH];
+  __shared__ float s_h[TC][GR_CH], s_b[TC][GR_CH];
   rl_pdl_trigger();
   const int ch = threadIdx.x % GR_CH, tc = threadIdx.x / GR_CH;
   const int c = blockIdx.x * GR_CH + ch;
@@ -78,34 +85,34 @@ gated_recurrence_kernel(const T* __restrict__ u, long long u_part, const float* 
   fetch(lo + tc * GR_STEPS);
   for (int t0 = lo; t0 < hi; t0 += TC * GR_STEPS) {
     const int first = t0 + tc * GR_STEPS;
-    float sa[GR_STEPS], sb[GR_STEPS], gy[GR_STEPS];
-    float A = 1.f, B = 0.f;
+    float sh[GR_STEPS], sb[GR_STEPS], gy[GR_STEPS];
+    float L = 0.f, B = 0.f;
 #pragma unroll
     for (int l = 0; l < GR_STEPS; ++l) {
-      sa[l] = 1.f; sb[l] = 0.f; gy[l] = 0.f;
+      sh[l] = 0.f; sb[l] = 0.f; gy[l] = 0.f;
       if (live && first + l < hi) {
-        const float2 s = gr_step(rl_ld(&ru[l]), rr[l] + br, ri[l] + bi, rate_sp);
-        sa[l] = s.x; sb[l] = s.y;
+        const GrStep s = gr_step(rl_ld(&ru[l]), rr[l] + br, ri[l] + bi, rate_sp);
+        sh[l] = s.h; sb[l] = s.b;
         gy[l] = gr_gelu(rl_ld(&ry[l]));
-        A *= s.x;
-        B = fmaf(s.x, B, s.y);
+        L += s.log_a;
+        B = gr_advance(B, s.h, s.b);
       }
     }
     if (t0 + TC * GR_STEPS < hi) fetch(first + TC * GR_STEPS);
     __syncthreads();                       // the previous span's steps have been read
-    s_a[tc][ch] = A;
+    s_h[tc][ch] = expm1f(L);
     s_b[tc][ch] = B;
     __syncthreads();
     float S = carry, mine = carry;
 #pragma unroll
     for (int j = 0; j < TC; ++j) {
       if (j == tc) mine = S;
-      S = fmaf(s_a[j][ch], S, s_b[j][ch]);
+      S = gr_advance(S, s_h[j][ch], s_b[j][ch]);
     }
     carry = S;
 #pragma unroll
     for (int l = 0; l < GR_STEPS; ++l) {
-      mine = fmaf(sa[l], mine, sb[l]);
+      mine = gr_advance(mine, sh[l], sb[l]);
       if (live && first + l < hi) rl_st(out + (size_t)(first + l) * ldo + c, mine * gy[l]);
     }
   }
@@ -189,10 +196,10 @@ gated_recurrence_step_kernel(const T* __restrict__ u, int ldu, const T* __restri
     const int c = blk * part + n;
     const int m = m0 + lane;
     const float rate_sp = rate * gr_softplus(lam[c]);
-    const float2 s = gr_step(s_in[lane * part + n], mr + z_bias[(size_t)blk * 2 * part + n], mi + z_bias[(size_t)blk * 2 * part + part + n],
+    const GrStep s = gr_step(s_in[lane * part + n], mr + z_bias[(size_t)blk * 2 * part + n], mi + z_bias[(size_t)blk * 2 * part + part + n],
                              rate_sp);
     float* st = state + (size_t)seq_slots[m] * state_stride + c;
-    const float S = fmaf(s.x, *st, s.y);
+    const float S = gr_advance(*st, s.h, s.b);
     *st = S;
     rl_st(out + (size_t)m * ldo + c, S * gr_gelu(rl_ld(y + (size_t)m * ldy + c)));
   }
