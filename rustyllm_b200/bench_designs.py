@@ -1,4 +1,4 @@
-"""Prompt and single-token throughput of the Mosurax, Mogutar and Forilorn designs beside the Llama decoder at equal layer sizes
+"""Prompt and single-token throughput of the Mosurax, Mogutar, Forilorn, Besuzen and Buketar designs beside the Llama decoder at equal layer sizes
 (random bfloat16 weights, synthetic tokens): ``python bench.py --designs`` or
 ``python -m rustyllm_b200.bench_designs [--size NAME] [--steps K] [--warmup W]``.
 
@@ -22,6 +22,11 @@ uses together with the shared one are as wide as the dense feed-forward), vocabu
                  decay a key channel (heads of 64, the model's width); the others rotated attention with an output gate an
                  element whose values are blended with the first such layer's; feed-forwards in turn dense (gelu on the gate)
                  and 16 experts in 4 groups (2 kept), 3 a token, softmax scores over all, with a gated shared expert
+  buketar        a residual of four streams; three layers in four a gated linear recurrence of the model's width with its gates
+                 in as many parts as heads, one in four attention through a latent (1/4 of the width, at most 512, plus a
+                 rotary key part of 64, queries straight from the input, a gate an element); every feed-forward 16
+                 experts, 4 a token, each a quarter of the dense width, sigmoid scores, clamped gates
+``--buketar-kernels`` times the Buketar design's kernels alone, each beside the like kernel of the closest designs.
 ``--besuzen-kernels`` times the Besuzen design's kernels alone, each beside the like kernel of the closest designs.
 ``--kernels`` times the Mogutar design's own kernels alone at the sizes of a layer (a JSON line a kernel, with the
 bytes it must move and their share of the measured copy bandwidth).
@@ -45,7 +50,7 @@ SIZES = {
                   experts=16, top=3, expert_ff=3584, shared_ff=3584),
 }
 MAX_POSITIONS = 4096
-MODELS = ("llama", "mosurax-dense", "mosurax-moe", "mogutar", "forilorn", "besuzen")
+MODELS = ("llama", "mosurax-dense", "mosurax-moe", "mogutar", "forilorn", "besuzen", "buketar")
 
 
 def llama_config(s: dict) -> dict:
@@ -119,6 +124,18 @@ def besuzen_config(s: dict) -> dict:
             "logit_scale": 0.5, "layers": layers}
 
 
+def buketar_config(s: dict, streams: int = 4) -> dict:
+    d, H, hd = s["width"], s["heads"], s["dim"]
+    rec = {"width": d, "blocks": H, "conv": 4}
+    lat = {"heads": H, "dim": hd, "rot_dim": 64, "vdim": hd, "kv_rank": min(512, d // 4), "scale": (hd + 64) ** -0.5,
+           "rot": {"base": 1.0e6, "dims": 64, "scaling": {"factor": 8.0, "original": 8192, "fast": 16.0, "slow": 2.0}}}
+    mlp = {"kind": "moe", "router": {"experts": s["experts"], "top": 4, "scale": 2.0}, "expert": {"ff": s["expert_ff"], "limit": 7.0}}
+    layers = [{"type": "latent_attention" if i % 4 == 2 else "rglru", "mixer": dict(lat if i % 4 == 2 else rec), "mlp": dict(mlp)}
+              for i in range(s["layers"])]
+    return {"architecture": "Buketar", "vocab": s["vocab"], "width": d, "norm": {"eps": 1e-5}, "streams": streams, "logit_softcap": 30.0,
+            "layers": layers}
+
+
 def measure(config: dict, prompt: int, batches: List[int], context: int, steps: int, warmup: int) -> Dict[str, float]:
     import numpy as np
     import torch
@@ -180,7 +197,7 @@ def run(sizes: List[str], prompt: int = 2048, batches=(8, 64), context: int = 10
         s = SIZES[name]
         got = {}
         for model in models:
-            cfg = llama_config(s) if model == "llama" else besuzen_config(s) if model == "besuzen" else mogutar_config(s, window or 1024) if model == "mogutar" \
+            cfg = llama_config(s) if model == "llama" else buketar_config(s) if model == "buketar" else besuzen_config(s) if model == "besuzen" else mogutar_config(s, window or 1024) if model == "mogutar" \
                 else forilorn_config(s, window or 1024) if model == "forilorn" else mosurax_config(s, model == "mosurax-moe", window or None)
             got[model] = measure(cfg, prompt, list(batches), context, steps, warmup)
             line = {"size": name, "model": model, "prompt_tokens": prompt, "context": context, "window": window or None,
@@ -640,6 +657,202 @@ def besuzen_kernel_times(sizes: List[str], prompt: int = 2048, batch: int = 64, 
     return lines
 
 
+class _KernelTimer:
+    """Times kernels alone (CUDA events, L2 flushed between runs, the median) and prints a JSON line each with the bytes
+    it must move, the operations it must do and the share of the roofline it reaches at the measured peaks."""
+
+    def __init__(self, runs: int):
+        import os
+        import torch
+        peaks = {}
+        try:
+            with open(os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "MEASURED_PEAKS.json")) as f:
+                peaks = json.load(f)
+        except OSError:
+            pass
+        self.gbs, self.tflops = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+        self.runs, self.lines = runs, []
+        self.dev = torch.device("cuda:0")
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device=self.dev)
+        self.e0, self.e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+
+    def timed(self, fn) -> float:
+        import torch
+        for _ in range(3):
+            fn()
+        ts = []
+        for _ in range(self.runs):
+            self.flush.zero_()
+            self.e0.record()
+            fn()
+            self.e1.record()
+            torch.cuda.synchronize()
+            ts.append(self.e0.elapsed_time(self.e1))
+        return sorted(ts)[len(ts) // 2] * 1e3   # us
+
+    def report(self, size, design, kernel, shape, fn, nbytes, flops=0.0) -> None:
+        us = self.timed(fn)
+        by_bytes, by_flops = nbytes / (self.gbs * 1e3), flops / (self.tflops * 1e6)
+        floor = max(by_bytes, by_flops)        # us
+        line = {"size": size, "design": design, "kernel": kernel, "shape": shape, "us": round(us, 2), "gb": round(nbytes / 1e9, 4),
+                "gflop": round(flops / 1e9, 3), "floor_us": round(floor, 2), "of_roofline": round(floor / us, 3),
+                "bound": "bandwidth" if by_bytes >= by_flops else "matrix"}
+        print(json.dumps(line), flush=True)
+        self.lines.append(line)
+
+
+def buketar_kernel_times(sizes: List[str], prompt: int = 2048, batch: int = 64, context: int = 1024, runs: int = 20) -> List[dict]:
+    """The Buketar design's kernels alone, each beside the like kernel of the closest designs (Mogutar: the norm that joins a
+    sublayer's output into the stream, recurrence, convolution, router, experts; Forilorn: the latent layer; Besuzen: products
+    of equal shape as one grouped product), bfloat16, at a layer's sizes: ``prompt`` tokens of one sequence, and one token of
+    each of ``batch`` sequences that hold ``context`` tokens with it."""
+    import torch
+    from . import kernels as K
+    from .cache.sequence_cache import KVNeed, SequenceCache
+    from .engine.step import StepState
+    t = _KernelTimer(runs)
+    dev, bf = t.dev, torch.bfloat16
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rnd = lambda *shape: torch.randn(shape, dtype=torch.float32, device=dev)
+    ones = lambda n: torch.ones(n, dtype=torch.float32, device=dev)
+
+    for name in sizes:
+        s = SIZES[name]
+        d, H, hd, E, F, S = s["width"], s["heads"], s["dim"], s["experts"], s["expert_ff"], 4
+        r, rd, qr = min(512, d // 4), 64, min(1536, 3 * d // 8)
+        for what, B, held, cnt in (("prompt", 1, 0, prompt), ("single tokens", batch, context - 1, 1)):
+            M = B * cnt
+            shape = f"{what}: {M} tokens, {B} seq of {held + cnt}"
+            cache = SequenceCache([KVNeed(1, r + rd, None, 0)], [None], 64 * (-(-(held + cnt) // 64) + 1) * B, bf, dev, max_slots=B)
+            slots = [cache.alloc_slot() for _ in range(B)]
+            if held:
+                cache.prepare(slots, [held] * B); cache.commit(slots, [held] * B)
+            cache.prepare(slots, [cnt] * B)
+            st = StepState(M, B, i32([0] * M), i32([held + k for _ in range(B) for k in range(cnt)]),
+                           i32([sl for sl in slots for _ in range(cnt)]), i32([cnt * b for b in range(B + 1)]), i32(slots),
+                           i32([held + cnt] * B), i32([]), [cnt] * B, [held + cnt] * B, cnt, held + cnt, cnt == 1)
+            group, layer = cache.kv_entry(0)
+            kp = group.k_pool(layer)
+            kp.normal_()
+            # ---- streams: a join with the next normed read, beside the norm that joins one stream ----
+            X, y, y1, w, xb = rnd(M, S, d), rnd(M, d), rnd(M, d), ones(d), torch.empty((M, d), dtype=bf, device=dev)
+            mix, to, coef = rnd(S, S) * 0.1, rnd(S), rnd(S)
+            t.report(name, "buketar", f"{S} streams joined, next normed read", f"{shape}, width {d}",
+                     lambda: K.streams_join(X, y, mix, to, w, coef=coef, norm_weight=w, eps=1e-5, out=xb), M * d * (8 * S + 4 + 2))
+            top = 4
+            rows, row, wts = rnd(M * top, d), torch.randperm(M * top, device=dev).to(torch.int32), torch.rand(M, top, device=dev)
+            t.report(name, "buketar", f"{S} streams joined from {top} experts' rows, next normed read", f"{shape}, width {d}",
+                     lambda: K.streams_join(X, rows, mix, to, w, row=row, weights=wts, coef=coef, norm_weight=w, eps=1e-5, out=xb),
+                     M * d * (8 * S + 4 * top + 2))
+            x = rnd(M, d)
+            t.report(name, "mogutar", "stream += norm(a + b) w, rounded copy", f"{shape}, width {d}",
+                     lambda: K.norm_add(x, y, 1.0, y1, 1.0, w, 1e-5, xb), M * d * (16 + 2))
+            res = torch.zeros_like(x)
+            del X
+            # ---- the recurrence ----
+            parts, n = H, d // H
+            proj = rnd(M, 2 * d).to(bf)
+            zb, lam = rnd(parts, 2 * n), rnd(d) - 4.0
+            rec = torch.zeros((B, 4 * d), dtype=torch.uint8, device=dev)
+            wg = (rnd(parts, 2 * n, n) * n ** -0.5).to(bf)
+            o = torch.empty((M, d), dtype=bf, device=dev)
+            if cnt == 1:
+                t.report(name, "buketar", "gates, recurrence, gelu branch", f"{shape}, width {d} in {parts} parts",
+                         lambda: K.gated_recurrence_step(proj[:, d:], wg, zb, lam, 8.0, proj[:, :d], o, rec, st.seq_slots),
+                         wg.numel() * 2 + M * d * (2 + 2 + 2 + 8), 4.0 * M * d * n)
+            else:
+                u, z = rnd(parts, M, n).to(bf), rnd(parts, M, 2 * n)
+                t.report(name, "buketar", "recurrence, gelu branch", f"{shape}, width {d}",
+                         lambda: K.gated_recurrence(u, z, zb, lam, 8.0, proj[:, :d], o, rec, st.cu_seqlens, st.seq_slots, st.q_lens),
+                         M * d * (2 + 8 + 2 + 2))
+                tile = K.gemm_tc_row_groups_tile(M)
+                t.report(name, "buketar", "gates' products, float out", f"{shape}, {parts} of {n} -> {2 * n}",
+                         lambda: K.gemm_tc_row_groups(u, wg, z, tile), M * d * (2 + 8) + wg.numel() * 2, 4.0 * M * d * n)
+                zh = z.to(bf)
+                t.report(name, "besuzen", "products of equal shape, bfloat16 out", f"{shape}, {parts} of {n} -> {2 * n}",
+                         lambda: K.gemm_tc_row_groups(u, wg, zh, tile), M * d * (2 + 4) + wg.numel() * 2, 4.0 * M * d * n)
+                del u, z, zh
+            Hr = d // 64
+            state = torch.zeros((B, 4 * Hr * 64 * 64), dtype=torch.uint8, device=dev)
+            qkv, o32 = rnd(M, 3 * d).to(bf), torch.empty((M, d), dtype=torch.float32, device=dev)
+            decay = torch.full((Hr,), 0.99, dtype=torch.float32, device=dev)
+            t.report(name, "mogutar", "linear attention with decay", f"{shape}, {Hr} heads of 64 x 64",
+                     lambda: K.linear_scan(qkv[:, :d], qkv[:, d:2 * d], qkv[:, 2 * d:], o32, state, st.cu_seqlens, st.seq_slots, Hr, 1, 64, 64,
+                                           decay, silu=True), qkv.numel() * 2 + o32.numel() * 4 + 2 * state.numel())
+            del qkv, o32, state
+            # ---- the filter in front ----
+            cw, cb = rnd(d, 4), rnd(d)
+            cs = torch.zeros((B, 4 * 3 * d), dtype=torch.uint8, device=dev)
+            moved = M * d * 4 + 2 * cs.numel()
+            if cnt == 1:
+                t.report(name, "buketar", "filter and its state, one kernel", f"{shape}, {d} channels, 4 taps",
+                         lambda: K.short_conv_step(proj[:, d:], cw, cb, False, st.seq_slots, cs, o), moved)
+            else:
+                up = torch.empty((parts, M, n), dtype=bf, device=dev)
+                t.report(name, "buketar", "filter in parts + state", f"{shape}, {d} channels, 4 taps",
+                         lambda: (K.short_conv(proj[:, d:], cw, cb, False, st.slot_of_token, cs, up),
+                                  K.short_conv_state(proj[:, d:], 4, st.cu_seqlens, st.seq_slots, cs)), moved)
+            t.report(name, "mogutar", "short convolution + state", f"{shape}, {d} channels, 4 taps",
+                     lambda: (K.short_conv(proj[:, d:], cw, cb, True, st.slot_of_token, cs, o),
+                              K.short_conv_state(proj[:, d:], 4, st.cu_seqlens, st.seq_slots, cs)), moved)
+            # ---- the latent layer ----
+            inv = torch.rand(rd // 2, dtype=torch.float32, device=dev)
+            pairs = sum(p + 1 for p in range(held, held + cnt)) * B
+            ql, ol = rnd(M, H * (r + rd)).to(bf), torch.empty((M, H * r), dtype=bf, device=dev)
+            hg = rnd(M, H).to(bf)
+            for design, kw in (("buketar", {}), ("forilorn", dict(gate=hg, gate_per_head=True))):
+                t.report(name, design, "attention over one latent row" + (", gate a head" if kw else ""),
+                         f"{shape}, {H} heads over rows of {r} + {rd}",
+                         lambda: K.attention(ql, kp, kp, group.page_table, st, ol, H, 1, r + rd, 0.07, value_dim=r, values_in_keys=True, **kw),
+                         (held + cnt) * B * (r + rd) * 2 + M * H * (2 * r + rd) * 2, 2.0 * pairs * H * (2 * r + rd))
+            q_cols = H * (hd + rd)
+            uw = rnd(M, q_cols + r + rd + H * hd).to(bf)
+            t.report(name, "buketar", "latent normed, rotary key (halves, magnitude), row to its page", f"{shape}, latent {r} + {rd}",
+                     lambda: K.latent_prepare(uw[:, q_cols:], 0, r, rd, None, ones(r), 1e-5, None, st.positions, st.slot_of_token,
+                                              group.page_table, inv, rd, False, kp, magnitude=1.2), M * 2 * (r + rd) * 2)
+            uf, cq = rnd(M, qr + r + rd + H).to(bf), torch.empty((M, qr), dtype=bf, device=dev)
+            t.report(name, "forilorn", "latents normed, rotary key (neighbours), row to its page", f"{shape}, latents {qr} and {r} + {rd}",
+                     lambda: K.latent_prepare(uf, qr, r, rd, ones(qr), ones(r), 1e-5, cq, st.positions, st.slot_of_token, group.page_table,
+                                              inv, rd, True, kp), M * (2 * qr + 2 * (r + rd)) * 2)
+            for design, inter, mag in (("buketar", False, 1.2), ("forilorn", True, 1.0)):
+                t.report(name, design, "query's rotary parts into place, " + ("neighbours" if inter else "halves, magnitude"),
+                         f"{shape}, {H} heads of {hd} + {rd}",
+                         lambda: K.latent_query(uw[:, :q_cols], ql, H, hd, rd, r, st.positions, inv, rd, inter, magnitude=mag), 2 * M * H * rd * 2)
+            wuv, ov = (rnd(H, hd, r) * r ** -0.5).to(bf), torch.empty((M, H * hd), dtype=bf, device=dev)
+            gates = uw[:, q_cols + r + rd:]
+            if cnt == 1:
+                for design, kw in (("buketar", dict(gate=gates)), ("forilorn", {})):
+                    t.report(name, design, "a product a head from the latent" + (", gate an element" if kw else ""), f"{shape}, {H} of {r} -> {hd}",
+                             lambda: K.heads_linear(ol, r, wuv, ov, hd, **kw), wuv.numel() * 2 + M * H * (r + hd * (2 if kw else 1)) * 2,
+                             2.0 * M * H * hd * r)
+            else:
+                t.report(name, "buketar", "output times sigmoid(gate), an element each", f"{shape}, {H * hd} columns",
+                         lambda: K.sigmoid_gate(ov, gates), M * H * hd * 6)
+            del cache, ql, ol, uw, uf
+            # ---- router and experts ----
+            h = rnd(M, d).to(bf)
+            wr = (rnd(E, d) * d ** -0.5).to(bf)
+            ids, wt = torch.empty((M, top), dtype=torch.int32, device=dev), torch.empty((M, top), dtype=torch.float32, device=dev)
+            logits = rnd(M, E)
+            for design, grp, keep, f in (("buketar", 1, 1, 2.0), ("mogutar", 4, 2, 1.0)):
+                if M < 128:
+                    fn = lambda: K.moe_route_scored(h, wr, None, top, grp, keep, ids, wt, softmax_all=False, group_top=2, renorm=False, weight_scale=f)
+                else:
+                    fn = lambda: K.moe_select_scored(logits, None, top, grp, keep, ids, wt, softmax_all=False, group_top=2, renorm=False, weight_scale=f)
+                t.report(name, design, ("router" if M < 128 else "choice from logits") + (", groups" if grp > 1 else ", factor"),
+                         f"{shape}, {E} experts", fn, (M * d * 2 + E * d * 2) if M < 128 else M * E * 4 + M * top * 8)
+            wgu, wd = (rnd(E, F, 2, d) * d ** -0.5).to(bf), (rnd(E, d, F) * F ** -0.5).to(bf)
+            used = min(E, M * top)
+            work = used * 3 * F * d * 2 + M * top * (2 * d + 2 * F + F) * 2 + M * top * d * 4
+            t.report(name, "buketar", "experts, clamped gate, rows left to the join", f"{shape}, {top} of {E}, {d} x {F}",
+                     lambda: K.moe_experts_grouped(h, wgu, wd, ids, wt, None, act=(7.0, 1.702)), work, 6.0 * M * top * F * d)
+            t.report(name, "mogutar", "experts, silu gate, added into the stream", f"{shape}, {top} of {E}, {d} x {F}",
+                     lambda: K.moe_experts_grouped(h, wgu, wd, ids, wt, res), work + M * d * 8 + M * top * d * 4, 6.0 * M * top * F * d)
+            del wgu, wd
+    K.check_device_errors()
+    return t.lines
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("--size", action="append", choices=sorted(SIZES), help="default: all")
@@ -649,6 +862,8 @@ def main(argv=None) -> int:
                     help="time the Forilorn design's kernels alone, each beside the like kernel of the Mosurax design, instead")
     ap.add_argument("--besuzen-kernels", action="store_true",
                     help="time the Besuzen design's kernels alone, each beside the like kernel of the Mosurax or Mogutar design, instead")
+    ap.add_argument("--buketar-kernels", action="store_true",
+                    help="time the Buketar design's kernels alone, each beside the like kernel of the closest designs, instead")
     ap.add_argument("--prompt", type=int, default=2048)
     ap.add_argument("--context", type=int, default=1024)
     ap.add_argument("--batch", type=int, action="append", help="default: 8 and 64")
@@ -661,6 +876,9 @@ def main(argv=None) -> int:
         return 0
     if a.besuzen_kernels:
         besuzen_kernel_times(a.size or sorted(SIZES), a.prompt, max(a.batch or (64,)), a.context)
+        return 0
+    if a.buketar_kernels:
+        buketar_kernel_times(a.size or sorted(SIZES), a.prompt, max(a.batch or (64,)), a.context)
         return 0
     if a.kernels:
         kernel_times(a.size or sorted(SIZES), a.prompt, max(a.batch or (64,)))
