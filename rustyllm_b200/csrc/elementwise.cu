@@ -483,6 +483,27 @@ __global__ void sigmoid_gate_kernel(T* __restrict__ y, int ldy, const T* __restr
   }
 }
 
+// rows that 16-byte accesses can fetch (bf16): a block a row, eight elements a thread at a time
+__global__ void __launch_bounds__(256)
+sigmoid_gate_rows_kernel(__nv_bfloat16* __restrict__ y, int ldy, const __nv_bfloat16* __restrict__ g, int ldg, int n) {
+  rl_pdl_trigger();
+  rl_pdl_wait();
+  __nv_bfloat16* yr = y + (size_t)blockIdx.x * ldy;
+  const __nv_bfloat16* gr = g + (size_t)blockIdx.x * ldg;
+  for (int i = 8 * threadIdx.x; i < n; i += 8 * 256) {
+    uint4 yv = *reinterpret_cast<const uint4*>(yr + i);
+    const uint4 gv = *reinterpret_cast<const uint4*>(gr + i);
+    __nv_bfloat162* yp = reinterpret_cast<__nv_bfloat162*>(&yv);
+    const __nv_bfloat162* gp = reinterpret_cast<const __nv_bfloat162*>(&gv);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float2 a = __bfloat1622float2(yp[k]), b = __bfloat1622float2(gp[k]);
+      yp[k] = __floats2bfloat162_rn(a.x * (1.0f / (1.0f + expf(-b.x))), a.y * (1.0f / (1.0f + expf(-b.y))));
+    }
+    *reinterpret_cast<uint4*>(yr + i) = yv;
+  }
+}
+
 extern "C" int rl_sigmoid_gate(void* y, int ldy, const void* g, int ldg, int dtype, int num_tokens, int n, cudaStream_t stream) {
   RL_REQUIRE(num_tokens >= 0 && n > 0 && ldy >= n && ldg >= n, "rl_sigmoid_gate: bad sizes M=%d n=%d", num_tokens, n);
   if (num_tokens == 0) return RL_OK;
@@ -490,7 +511,9 @@ extern "C" int rl_sigmoid_gate(void* y, int ldy, const void* g, int ldg, int dty
   const int threads = 256;
   const size_t want = (total + threads - 1) / threads;
   const int blocks = (int)(want < (size_t)rl_num_sms() * 16 ? want : (size_t)rl_num_sms() * 16);
-  if (dtype == RL_F32)
+  if (dtype == RL_BF16 && n % 8 == 0 && ldy % 8 == 0 && ldg % 8 == 0 && (((uintptr_t)y | (uintptr_t)g) & 15) == 0)
+    rl_launch_pdl(sigmoid_gate_rows_kernel, num_tokens, 256, 0, stream, (__nv_bfloat16*)y, ldy, (const __nv_bfloat16*)g, ldg, n);
+  else if (dtype == RL_F32)
     rl_launch_pdl(sigmoid_gate_kernel<float>, blocks, threads, 0, stream, (float*)y, ldy, (const float*)g, ldg, num_tokens, n);
   else if (dtype == RL_BF16)
     rl_launch_pdl(sigmoid_gate_kernel<__nv_bfloat16>, blocks, threads, 0, stream, (__nv_bfloat16*)y, ldy, (const __nv_bfloat16*)g, ldg, num_tokens, n);

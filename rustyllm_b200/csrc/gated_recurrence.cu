@@ -16,13 +16,15 @@
 //                            reduces them to one step of the same form, the threads' steps are composed in order
 //                            through shared memory, and each replays its tokens from its own start.
 // rl_gated_recurrence_step   one token a sequence: the gates' products, the recurrence and the output in one kernel.
-//                            A warp owns a channel (its row of either matrix) for 16 tokens whose inputs wait in
-//                            shared memory; the lane that ends up with a token's sums advances its state.
+//                            bfloat16: a block takes 16 channels (32 matrix rows) for up to 64 tokens on the tensor
+//                            cores.  Any shape: a warp owns a channel for 16 tokens whose inputs wait in shared
+//                            memory; the lane that ends up with a token's sums advances its state.
 // rl_short_conv_step         the causal filter in front, one token a sequence: filter and shift of the kept inputs
 //                            in one kernel (a thread owns a channel of a sequence, so nobody else reads them).
 #include <math.h>
 
 #include "common.cuh"
+#include "small_product.cuh"
 
 #define GR_CH 16
 #define GR_STEPS 8
@@ -35,11 +37,34 @@ __device__ __forceinline__ float gr_gelu(float z) {
 }
 // the token's step of the recurrence: S -> S + (h S + b); log a
 struct GrStep { float log_a, h, b; };
+// A 32-bit run takes the accurate functions; a bfloat16 run (whose inputs carry 8 bits and whose kernel would be bound by
+// instructions) the fast exponential, division and reciprocal square root, and e^x - 1 near 0 by the first terms of its
+// power series: all of them float and good to about 2^-20.
+template <typename T> struct GrMath;
+template <> struct GrMath<float> {
+  static __device__ __forceinline__ float sigmoid(float z) { return gr_sigmoid(z); }
+  static __device__ __forceinline__ float expm1(float x) { return expm1f(x); }
+  static __device__ __forceinline__ float root(float x) { return sqrtf(x); }
+  static __device__ __forceinline__ float gelu(float z) { return gr_gelu(z); }
+};
+template <> struct GrMath<__nv_bfloat16> {
+  static __device__ __forceinline__ float sigmoid(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
+  static __device__ __forceinline__ float expm1(float x) {      // x <= 0; the series' next term is below 2^-20 of x up to |x| = 1/4
+    const float near0 = x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.0f / 120.0f, 1.0f / 24.0f), 1.0f / 6.0f), 0.5f), 1.0f);
+    return x > -0.25f ? near0 : __expf(x) - 1.0f;
+  }
+  static __device__ __forceinline__ float root(float x) { return x * rsqrtf(fmaxf(x, 1e-37f)); }
+  static __device__ __forceinline__ float gelu(float z) {       // z / (1 + e^{-2y}), y the argument of the tanh
+    const float y = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+    return __fdividef(z, 1.0f + __expf(fminf(-2.0f * y, 80.0f)));
+  }
+};
+template <typename T>
 __device__ __forceinline__ GrStep gr_step(float u, float zr, float zi, float rate_sp) {
   GrStep s;
-  s.log_a = -rate_sp * gr_sigmoid(zr);
-  s.h = expm1f(s.log_a);
-  s.b = sqrtf(-s.h * (2.0f + s.h)) * gr_sigmoid(zi) * u;
+  s.log_a = -rate_sp * GrMath<T>::sigmoid(zr);
+  s.h = GrMath<T>::expm1(s.log_a);
+  s.b = GrMath<T>::root(-s.h * (2.0f + s.h)) * GrMath<T>::sigmoid(zi) * u;
   return s;
 }
 __device__ __forceinline__ float gr_advance(float S, float h, float b) { return S + fmaf(h, S, b); }
@@ -52,7 +77,8 @@ gated_recurrence_kernel(const T* __restrict__ u, long long u_part, const float* 
                         const float* __restrict__ z_bias, const float* __restrict__ lam, float rate, const T* __restrict__ y, int ldy,
                         T* __restrict__ out, int ldo, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slots,
                         float* __restrict__ state, long long state_stride, int W, int part) {
-  __shared__ float s_h[TC][GR_CH], s_b[TC][GR_CH];
+  static_assert(GR_CH == 16, "a warp holds two runs of tokens of the same channels");
+  __shared__ float s_h[2][TC / 2][GR_CH], s_b[2][TC / 2][GR_CH];      // a pair of runs as one step; two spans in turn
   rl_pdl_trigger();
   const int ch = threadIdx.x % GR_CH, tc = threadIdx.x / GR_CH;
   const int c = blockIdx.x * GR_CH + ch;
@@ -83,7 +109,8 @@ gated_recurrence_kernel(const T* __restrict__ u, long long u_part, const float* 
     }
   };
   fetch(lo + tc * GR_STEPS);
-  for (int t0 = lo; t0 < hi; t0 += TC * GR_STEPS) {
+  int buf = 0;
+  for (int t0 = lo; t0 < hi; t0 += TC * GR_STEPS, buf ^= 1) {
     const int first = t0 + tc * GR_STEPS;
     float sh[GR_STEPS], sb[GR_STEPS], gy[GR_STEPS];
     float L = 0.f, B = 0.f;
@@ -91,25 +118,32 @@ gated_recurrence_kernel(const T* __restrict__ u, long long u_part, const float* 
     for (int l = 0; l < GR_STEPS; ++l) {
       sh[l] = 0.f; sb[l] = 0.f; gy[l] = 0.f;
       if (live && first + l < hi) {
-        const GrStep s = gr_step(rl_ld(&ru[l]), rr[l] + br, ri[l] + bi, rate_sp);
+        const GrStep s = gr_step<T>(rl_ld(&ru[l]), rr[l] + br, ri[l] + bi, rate_sp);
         sh[l] = s.h; sb[l] = s.b;
-        gy[l] = gr_gelu(rl_ld(&ry[l]));
+        gy[l] = GrMath<T>::gelu(rl_ld(&ry[l]));
         L += s.log_a;
         B = gr_advance(B, s.h, s.b);
       }
     }
     if (t0 + TC * GR_STEPS < hi) fetch(first + TC * GR_STEPS);
-    __syncthreads();                       // the previous span's steps have been read
-    s_h[tc][ch] = expm1f(L);
-    s_b[tc][ch] = B;
+    // the two runs of a warp joined, then the pairs in order.  (A buffer is written again two spans later; the barrier of
+    // the span between has seen every reader leave.)
+    const float h = GrMath<T>::expm1(L);
+    const float oL = __shfl_xor_sync(0xffffffffu, L, GR_CH), oh = __shfl_xor_sync(0xffffffffu, h, GR_CH);
+    const float oB = __shfl_xor_sync(0xffffffffu, B, GR_CH);
+    if (tc & 1) {
+      s_h[buf][tc >> 1][ch] = GrMath<T>::expm1(L + oL);
+      s_b[buf][tc >> 1][ch] = gr_advance(oB, h, B);
+    }
     __syncthreads();
     float S = carry, mine = carry;
 #pragma unroll
-    for (int j = 0; j < TC; ++j) {
-      if (j == tc) mine = S;
-      S = gr_advance(S, s_h[j][ch], s_b[j][ch]);
+    for (int j = 0; j < TC / 2; ++j) {
+      if (j == tc >> 1) mine = S;
+      S = gr_advance(S, s_h[buf][j][ch], s_b[buf][j][ch]);
     }
     carry = S;
+    if (tc & 1) mine = gr_advance(mine, oh, oB);
 #pragma unroll
     for (int l = 0; l < GR_STEPS; ++l) {
       mine = gr_advance(mine, sh[l], sb[l]);
@@ -196,13 +230,90 @@ gated_recurrence_step_kernel(const T* __restrict__ u, int ldu, const T* __restri
     const int c = blk * part + n;
     const int m = m0 + lane;
     const float rate_sp = rate * gr_softplus(lam[c]);
-    const GrStep s = gr_step(s_in[lane * part + n], mr + z_bias[(size_t)blk * 2 * part + n], mi + z_bias[(size_t)blk * 2 * part + part + n],
+    const GrStep s = gr_step<T>(s_in[lane * part + n], mr + z_bias[(size_t)blk * 2 * part + n], mi + z_bias[(size_t)blk * 2 * part + part + n],
                              rate_sp);
     float* st = state + (size_t)seq_slots[m] * state_stride + c;
     const float S = gr_advance(*st, s.h, s.b);
     *st = S;
-    rl_st(out + (size_t)m * ldo + c, S * gr_gelu(rl_ld(y + (size_t)m * ldy + c)));
+    rl_st(out + (size_t)m * ldo + c, S * GrMath<T>::gelu(rl_ld(y + (size_t)m * ldy + c)));
   }
+}
+
+#define GR_MMA_CH (SP_ROWS / 2)
+template <int TW>
+__global__ void __launch_bounds__(SP_THREADS)
+gated_recurrence_step_mma_kernel(const __nv_bfloat16* __restrict__ u, int ldu, const __nv_bfloat16* __restrict__ w,
+                                 const float* __restrict__ z_bias, const float* __restrict__ lam, float rate,
+                                 const __nv_bfloat16* __restrict__ y, int ldy, __nv_bfloat16* __restrict__ out, int ldo,
+                                 const int* __restrict__ seq_slots, float* __restrict__ state, long long state_stride, int M, int part) {
+  extern __shared__ __align__(128) uint8_t gr_smem[];
+  rl_pdl_trigger();
+  const SpLayout L = sp_layout(part, TW);
+  const int blk = blockIdx.y, n0 = blockIdx.x * GR_MMA_CH, m0 = blockIdx.z * 16 * TW;
+  const int chans = min(GR_MMA_CH, part - n0), toks = min(16 * TW, M - m0);
+  // rows 0 .. 15: the channels' decay-gate rows, 16 .. 31: their input-gate rows (a row beyond the part repeats a live one)
+  const __nv_bfloat16* wb = w + (size_t)blk * 2 * part * part;
+  sp_fetch(gr_smem, 0, SP_ROWS, SP_ROWS, part, L, [&](int r) {
+    const int ch = min(r % GR_MMA_CH, chans - 1);
+    return wb + (size_t)((r / GR_MMA_CH) * part + n0 + ch) * part;
+  });
+  const int ch = threadIdx.x % GR_MMA_CH;
+  const bool live = ch < chans;
+  const int c = blk * part + n0 + (live ? ch : 0);
+  const float rate_sp = rate * gr_softplus(lam[c]);
+  const float br = z_bias[(size_t)blk * 2 * part + n0 + (live ? ch : 0)];
+  const float bi = z_bias[(size_t)blk * 2 * part + part + n0 + (live ? ch : 0)];
+  rl_pdl_wait();
+  sp_fetch(gr_smem, L.x_off, 16 * TW, toks, part, L, [&](int r) { return u + (size_t)(m0 + r) * ldu + (size_t)blk * part; });
+  sp_commit();
+  // what the epilogue needs besides the sums, requested beside the operands
+  constexpr int PER = 16 * TW * GR_MMA_CH / SP_THREADS;      // (token, channel) pairs a thread
+  float S[PER], yv[PER];
+  float* st[PER];
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int m = threadIdx.x / GR_MMA_CH + i * (SP_THREADS / GR_MMA_CH);
+    S[i] = yv[i] = 0.f;
+    st[i] = nullptr;
+    if (live && m < toks) {
+      st[i] = state + (size_t)seq_slots[m0 + m] * state_stride + c;
+      S[i] = *st[i];
+      yv[i] = __bfloat162float(y[(size_t)(m0 + m) * ldy + c]);
+    }
+  }
+  sp_wait_all();
+  __syncthreads();
+  sp_multiply<TW>(gr_smem, L);
+  const __nv_bfloat16* s_u = reinterpret_cast<const __nv_bfloat16*>(gr_smem + L.x_off);
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int m = threadIdx.x / GR_MMA_CH + i * (SP_THREADS / GR_MMA_CH);
+    if (st[i] == nullptr) continue;
+    const GrStep s = gr_step<__nv_bfloat16>(__bfloat162float(s_u[m * L.ld + n0 + ch]), sp_sum<TW>(gr_smem, L, ch, m) + br,
+                                            sp_sum<TW>(gr_smem, L, GR_MMA_CH + ch, m) + bi, rate_sp);
+    const float next = gr_advance(S[i], s.h, s.b);
+    *st[i] = next;
+    out[(size_t)(m0 + m) * ldo + c] = __float2bfloat16_rn(next * GrMath<__nv_bfloat16>::gelu(yv[i]));
+  }
+}
+
+template <int TW>
+static int gr_step_mma(const void* u, int ldu, const void* w, const float* z_bias, const float* lam, float rate, const void* y, int ldy,
+                       void* out, int ldo, const int* seq_slots, int num_seqs, float* state, long long state_stride, int width, int part,
+                       cudaStream_t stream) {
+  const SpLayout L = sp_layout(part, TW);
+  static int reserved = 48 * 1024;
+  if ((int)L.bytes > reserved) {
+    cudaError_t e = cudaFuncSetAttribute(gated_recurrence_step_mma_kernel<TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L.bytes);
+    RL_REQUIRE(e == cudaSuccess, "rl_gated_recurrence_step: cannot reserve %u bytes of shared memory: %s", L.bytes, cudaGetErrorString(e));
+    reserved = (int)L.bytes;
+  }
+  const dim3 grid((part + GR_MMA_CH - 1) / GR_MMA_CH, width / part, (num_seqs + 16 * TW - 1) / (16 * TW));
+  rl_launch_pdl(gated_recurrence_step_mma_kernel<TW>, grid, dim3(SP_THREADS), L.bytes, stream, (const __nv_bfloat16*)u, ldu,
+                (const __nv_bfloat16*)w, z_bias, lam, rate, (const __nv_bfloat16*)y, ldy, (__nv_bfloat16*)out, ldo, seq_slots, state,
+                state_stride, num_seqs, part);
+  RL_LAUNCH_CHECK("rl_gated_recurrence_step");
+  return RL_OK;
 }
 
 // state: kept inputs float [taps - 1, C] a slot, oldest first (as rl_short_conv).  A fresh slot's are zero.
@@ -300,6 +411,16 @@ extern "C" int rl_gated_recurrence_step(const void* u, int ldu, const void* w, c
              rl_gated_recurrence_step_max_part());
   RL_REQUIRE(ldu >= width && ldy >= width && ldo >= width, "rl_gated_recurrence_step: row strides too small");
   if (num_seqs == 0) return RL_OK;
+  if (dtype == RL_BF16 && part % 8 == 0 && ldu % 8 == 0 && (((uintptr_t)u | (uintptr_t)w) & 15) == 0 && num_seqs <= 65535 * 16 &&
+      sp_layout(part, sp_token_warps(num_seqs)).bytes <= 200u * 1024u) {
+#define RL_GM(TW) gr_step_mma<TW>(u, ldu, w, z_bias, lam, rate, y, ldy, out, ldo, seq_slots, num_seqs, state, state_stride, width, part, stream)
+    switch (sp_token_warps(num_seqs)) {
+      case 1: return RL_GM(1);
+      case 2: return RL_GM(2);
+      default: return RL_GM(4);
+    }
+#undef RL_GM
+  }
   const dim3 grid((part + 7) / 8, width / part, (num_seqs + GR_STEP_TOKENS - 1) / GR_STEP_TOKENS);
   RL_REQUIRE(grid.z <= 65535, "rl_gated_recurrence_step: too many sequences (%d)", num_seqs);
   const size_t smem = (size_t)GR_STEP_TOKENS * part * sizeof(float);

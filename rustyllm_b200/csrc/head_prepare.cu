@@ -17,6 +17,7 @@
 #include <math.h>
 
 #include "common.cuh"
+#include "small_product.cuh"
 
 #define HP_WARPS 4
 #define HP_MAX_W 256
@@ -487,6 +488,51 @@ heads_linear_kernel(const T* __restrict__ x, int ldx, int x_head, const T* __res
   }
 }
 
+// The same on the tensor cores (bf16, rows that 16-byte copies can fetch): 32 output columns of one head for up to 64
+// tokens a block.
+template <int TW>
+__global__ void __launch_bounds__(SP_THREADS)
+heads_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int x_head, const __nv_bfloat16* __restrict__ w,
+                        __nv_bfloat16* __restrict__ out, int ldo, int out_head, int M, int N, int K,
+                        const __nv_bfloat16* __restrict__ gate, int ldg) {
+  extern __shared__ __align__(128) uint8_t hl_smem[];
+  rl_pdl_trigger();
+  const SpLayout L = sp_layout(K, TW);
+  const int a = blockIdx.y, n0 = blockIdx.x * SP_ROWS, m0 = blockIdx.z * 16 * TW;
+  const int rows = min(SP_ROWS, N - n0), toks = min(16 * TW, M - m0);
+  sp_fetch(hl_smem, 0, SP_ROWS, rows, K, L, [&](int r) { return w + ((size_t)a * N + n0 + r) * K; });      // no kernel of a step writes weights
+  rl_pdl_wait();
+  sp_fetch(hl_smem, L.x_off, 16 * TW, toks, K, L, [&](int r) { return x + (size_t)(m0 + r) * ldx + (size_t)a * x_head; });
+  sp_commit();
+  sp_wait_all();
+  __syncthreads();
+  sp_multiply<TW>(hl_smem, L);
+  const int lane = threadIdx.x & 31;
+  if (lane >= rows) return;
+  for (int m = threadIdx.x >> 5; m < toks; m += SP_THREADS / 32) {
+    float v = sp_sum<TW>(hl_smem, L, lane, m);
+    if (gate) v *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)(m0 + m) * ldg + (size_t)a * N + n0 + lane])));
+    out[(size_t)(m0 + m) * ldo + (size_t)a * out_head + n0 + lane] = __float2bfloat16_rn(v);
+  }
+}
+
+template <int TW>
+static int heads_linear_mma(const void* x, int ldx, int x_head, const void* w, void* out, int ldo, int out_head, int M, int H, int N, int K,
+                            const void* gate, int ldg, cudaStream_t stream) {
+  const SpLayout L = sp_layout(K, TW);
+  static int reserved = 48 * 1024;
+  if ((int)L.bytes > reserved) {
+    cudaError_t e = cudaFuncSetAttribute(heads_linear_mma_kernel<TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L.bytes);
+    RL_REQUIRE(e == cudaSuccess, "rl_heads_linear: cannot reserve %u bytes of shared memory: %s", L.bytes, cudaGetErrorString(e));
+    reserved = (int)L.bytes;
+  }
+  const dim3 grid((N + SP_ROWS - 1) / SP_ROWS, H, (M + 16 * TW - 1) / (16 * TW));
+  rl_launch_pdl(heads_linear_mma_kernel<TW>, grid, dim3(SP_THREADS), L.bytes, stream, (const __nv_bfloat16*)x, ldx, x_head,
+                (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, out_head, M, N, K, (const __nv_bfloat16*)gate, ldg);
+  RL_LAUNCH_CHECK("rl_heads_linear");
+  return RL_OK;
+}
+
 // x: [M, ldx] with head a's K inputs at columns [a * x_head, a * x_head + K); w: [H, N, K] contiguous; out: [M, ldo]
 // with head a's N outputs at columns [a * out_head, a * out_head + N); all of one dtype, sums in 32-bit.  gate (may be
 // null): [M, ldg] with head a's N values at columns [a * N, a * N + N); an output is multiplied by its sigmoid.
@@ -496,6 +542,14 @@ extern "C" int rl_heads_linear(const void* x, int ldx, int x_head, const void* w
   RL_REQUIRE(ldx >= (H - 1) * x_head + K && ldo >= (H - 1) * out_head + N && x_head >= 0 && out_head >= N,
              "rl_heads_linear: row strides too small for the heads");
   RL_REQUIRE(gate == nullptr || ldg >= H * N, "rl_heads_linear: the gate's row stride is too small");
+  if (M > 0 && dtype == RL_BF16 && K % 8 == 0 && x_head % 8 == 0 && ldx % 8 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0 &&
+      sp_layout(K, sp_token_warps(M)).bytes <= 200u * 1024u && (M + 63) / 64 <= 65535) {
+    switch (sp_token_warps(M)) {
+      case 1: return heads_linear_mma<1>(x, ldx, x_head, w, out, ldo, out_head, M, H, N, K, gate, ldg, stream);
+      case 2: return heads_linear_mma<2>(x, ldx, x_head, w, out, ldo, out_head, M, H, N, K, gate, ldg, stream);
+      default: return heads_linear_mma<4>(x, ldx, x_head, w, out, ldo, out_head, M, H, N, K, gate, ldg, stream);
+    }
+  }
   const size_t smem = (size_t)HL_TOKENS * K * sizeof(float);
   RL_REQUIRE(smem <= 48 * 1024, "rl_heads_linear: %d inputs a head exceed the %d this kernel holds", K, 48 * 1024 / (HL_TOKENS * 4));
   if (M == 0) return RL_OK;

@@ -74,6 +74,69 @@ short_conv_kernel(const T* __restrict__ u, int ldu, const float* __restrict__ w,
   rl_st(out + (size_t)(c / part) * out_part + (size_t)m * ldo + c % part, acc);
 }
 
+// The same for many tokens: a thread takes V neighbouring channels of CONV_RUN consecutive rows and keeps the last
+// taps - 1 inputs in registers, so an input is loaded once a run instead of once a tap.  Only where a row opens another
+// sequence (or the run) are the predecessors looked up.  Sums run in the same order as above.
+#define CONV_RUN 8
+template <typename T, int V> struct __align__(8) ConvVec { T v[V]; };
+template <typename T, int V, int TAPS>
+__global__ void __launch_bounds__(128)
+short_conv_run_kernel(const T* __restrict__ u, int ldu, const float* __restrict__ w, const float* __restrict__ bias, int act, int C,
+                      const int* __restrict__ slot_of_token, const float* __restrict__ state, long long state_stride,
+                      T* __restrict__ out, int ldo, int part, long long out_part, int M) {
+  rl_pdl_trigger();
+  const int c = V * (blockIdx.y * 128 + threadIdx.x);
+  if (c >= C) return;
+  float f[V][TAPS], b[V];
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    b[k] = bias ? bias[c + k] : 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) f[k][j] = w[(size_t)(c + k) * TAPS + j];
+  }
+  rl_pdl_wait();
+  const int m0 = blockIdx.x * CONV_RUN, rows = min(CONV_RUN, M - m0);
+  T* o = out + (size_t)(c / part) * out_part + c % part;
+  ConvVec<T, V> in[CONV_RUN];
+  int slots[CONV_RUN];
+#pragma unroll
+  for (int r = 0; r < CONV_RUN; ++r)
+    if (r < rows) {
+      in[r] = *reinterpret_cast<const ConvVec<T, V>*>(u + (size_t)(m0 + r) * ldu + c);
+      slots[r] = slot_of_token[m0 + r];
+    }
+  float hist[V][TAPS];                   // hist[k][j]: the input TAPS - 1 - j positions back; [TAPS - 1] is the row's own
+#pragma unroll
+  for (int r = 0; r < CONV_RUN; ++r) {
+    if (r >= rows) break;
+    const int m = m0 + r;
+    if (r == 0 || slots[r] != slots[r > 0 ? r - 1 : 0]) {
+      const int n = r == 0 ? conv_rows_back(slot_of_token, m, TAPS) : 0;
+      const float* st = state + (size_t)slots[r] * state_stride;
+#pragma unroll
+      for (int k = 0; k < V; ++k)
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) hist[k][j] = conv_input(u, ldu, st, C, TAPS, m, n, TAPS - 1 - j, c + k);
+    } else {
+#pragma unroll
+      for (int k = 0; k < V; ++k)
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) hist[k][j] = hist[k][j + 1];
+    }
+    ConvVec<T, V> res;
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      hist[k][TAPS - 1] = rl_ld(&in[r].v[k]);
+      float acc = b[k];
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) acc = fmaf(f[k][j], hist[k][j], acc);
+      if (act == 1) acc = acc / (1.0f + expf(-acc));
+      rl_st(&res.v[k], acc);
+    }
+    *reinterpret_cast<ConvVec<T, V>*>(o + (size_t)m * ldo) = res;
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(CONV_THREADS)
 short_conv_state_kernel(const T* __restrict__ u, int ldu, int C, int taps, const int* __restrict__ cu_seqlens,
@@ -200,6 +263,28 @@ extern "C" int rl_short_conv_parts(const void* u, int ldu, int dtype, const floa
   RL_REQUIRE(ldu >= channels && ldo >= part, "rl_short_conv: row strides too small");
   RL_REQUIRE(act == 0 || act == 1, "rl_short_conv: unknown activation %d", act);
   if (num_tokens == 0) return RL_OK;
+  // four bf16 channels (8 bytes) or two float ones a thread where the rows allow it and there are tokens enough
+  const uintptr_t bits = (uintptr_t)u | (uintptr_t)out;
+  if (num_tokens >= 128 && taps >= 2 && taps <= 4 && channels % 4 == 0 && part % 4 == 0 && ldu % 4 == 0 && ldo % 4 == 0 && out_part % 4 == 0 &&
+      (bits & 7) == 0 && (dtype == RL_BF16 || dtype == RL_F32)) {
+    const int V = dtype == RL_BF16 ? 4 : 2;
+    const dim3 g((num_tokens + CONV_RUN - 1) / CONV_RUN, (channels / V + 127) / 128);
+#define RL_CONV_RUN(T, VV, TAPS)                                                                                                  \
+  rl_launch_pdl(short_conv_run_kernel<T, VV, TAPS>, g, dim3(128), 0, stream, (const T*)u, ldu, w, bias, act, channels, slot_of_token, \
+                state, state_stride, (T*)out, ldo, part, out_part, num_tokens)
+    if (dtype == RL_BF16) {
+      if (taps == 2) RL_CONV_RUN(__nv_bfloat16, 4, 2);
+      else if (taps == 3) RL_CONV_RUN(__nv_bfloat16, 4, 3);
+      else RL_CONV_RUN(__nv_bfloat16, 4, 4);
+    } else {
+      if (taps == 2) RL_CONV_RUN(float, 2, 2);
+      else if (taps == 3) RL_CONV_RUN(float, 2, 3);
+      else RL_CONV_RUN(float, 2, 4);
+    }
+#undef RL_CONV_RUN
+    RL_LAUNCH_CHECK("rl_short_conv");
+    return RL_OK;
+  }
   const dim3 grid(num_tokens, (channels + CONV_THREADS - 1) / CONV_THREADS);
   if (dtype == RL_F32)
     rl_launch_pdl(short_conv_kernel<float>, grid, CONV_THREADS, 0, stream, (const float*)u, ldu, w, bias, act, channels, taps,
