@@ -27,7 +27,7 @@
 #include "small_product.cuh"
 
 #define GR_CH 16
-#define GR_STEPS 8
+#define GR_STEPS 4
 #define GR_STEP_TOKENS 16
 
 __device__ __forceinline__ float gr_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
@@ -72,7 +72,7 @@ __device__ __forceinline__ float gr_advance(float S, float h, float b) { return 
 // u: channel c of token m at u[(c / part) * u_part + m * part + c % part]; z: float, its two sums at
 // z[(c / part) * z_part + m * 2 part + c % part] (decay gate) and + part (input gate).
 template <typename T, int TC>
-__global__ void __launch_bounds__(GR_CH * TC)
+__global__ void __launch_bounds__(GR_CH * TC, TC > 8 ? 2 : 1)
 gated_recurrence_kernel(const T* __restrict__ u, long long u_part, const float* __restrict__ z, long long z_part,
                         const float* __restrict__ z_bias, const float* __restrict__ lam, float rate, const T* __restrict__ y, int ldy,
                         T* __restrict__ out, int ldo, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slots,
@@ -89,9 +89,11 @@ gated_recurrence_kernel(const T* __restrict__ u, long long u_part, const float* 
   rl_pdl_wait();
   const int b = blockIdx.y;
   const int lo = cu_seqlens[b], hi = cu_seqlens[b + 1];
+  if (lo >= hi) return;
   float* st = state + (size_t)seq_slots[b] * state_stride;
   const T* up = u + (size_t)blk * u_part + at;
   const float* zp = z + (size_t)blk * z_part + at;
+  const T* yp = y + (live ? c : 0);
   float carry = live ? st[c] : 0.f;
   // a token's three inputs are requested one span ahead
   T ru[GR_STEPS], ry[GR_STEPS];
@@ -99,13 +101,11 @@ gated_recurrence_kernel(const T* __restrict__ u, long long u_part, const float* 
   auto fetch = [&](int first) {
 #pragma unroll
     for (int l = 0; l < GR_STEPS; ++l) {
-      const int m = first + l;
-      if (live && m < hi) {
-        ru[l] = up[(size_t)m * part];
-        rr[l] = zp[(size_t)m * 2 * part];
-        ri[l] = zp[(size_t)m * 2 * part + part];
-        ry[l] = y[(size_t)m * ldy + c];
-      }
+      const int m = min(first + l, hi - 1);          // (a row behind the last one is loaded and not used)
+      ru[l] = up[(size_t)m * part];
+      rr[l] = zp[(size_t)m * 2 * part];
+      ri[l] = zp[(size_t)m * 2 * part + part];
+      ry[l] = yp[(size_t)m * ldy];
     }
   };
   fetch(lo + tc * GR_STEPS);
@@ -116,14 +116,13 @@ gated_recurrence_kernel(const T* __restrict__ u, long long u_part, const float* 
     float L = 0.f, B = 0.f;
 #pragma unroll
     for (int l = 0; l < GR_STEPS; ++l) {
-      sh[l] = 0.f; sb[l] = 0.f; gy[l] = 0.f;
-      if (live && first + l < hi) {
-        const GrStep s = gr_step<T>(rl_ld(&ru[l]), rr[l] + br, ri[l] + bi, rate_sp);
-        sh[l] = s.h; sb[l] = s.b;
-        gy[l] = GrMath<T>::gelu(rl_ld(&ry[l]));
-        L += s.log_a;
-        B = gr_advance(B, s.h, s.b);
-      }
+      const bool valid = first + l < hi;             // no branch: the steps' long chains overlap
+      const GrStep s = gr_step<T>(rl_ld(&ru[l]), rr[l] + br, ri[l] + bi, rate_sp);
+      sh[l] = valid ? s.h : 0.f;
+      sb[l] = valid ? s.b : 0.f;
+      gy[l] = GrMath<T>::gelu(rl_ld(&ry[l]));
+      L += valid ? s.log_a : 0.f;
+      B = gr_advance(B, sh[l], sb[l]);
     }
     if (t0 + TC * GR_STEPS < hi) fetch(first + TC * GR_STEPS);
     // the two runs of a warp joined, then the pairs in order.  (A buffer is written again two spans later; the barrier of
@@ -384,7 +383,7 @@ extern "C" int rl_gated_recurrence(const void* u, long long u_part, const float*
 #define RL_GR(T, TC)                                                                                                              \
   rl_launch_pdl(gated_recurrence_kernel<T, TC>, grid, dim3(GR_CH * TC), 0, stream, (const T*)u, u_part, z, z_part, z_bias, lam, rate, \
                 (const T*)y, ldy, (T*)out, ldo, cu_seqlens, seq_slots, state, state_stride, width, part)
-  const bool many = longest > 4 * GR_STEPS;
+  const bool many = longest > 8 * GR_STEPS;
   if (dtype == RL_F32) {
     if (many) RL_GR(float, 32); else RL_GR(float, 4);
   } else if (dtype == RL_BF16) {

@@ -504,14 +504,26 @@ heads_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int x_head
   rl_pdl_wait();
   sp_fetch(hl_smem, L.x_off, 16 * TW, toks, K, L, [&](int r) { return x + (size_t)(m0 + r) * ldx + (size_t)a * x_head; });
   sp_commit();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  constexpr int PER = 16 * TW / (SP_THREADS / 32);           // tokens a warp finishes
+  __nv_bfloat16 gv[PER];
+  if (gate) {                                                 // requested beside the operands
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int m = min(warp + i * (SP_THREADS / 32), toks - 1);
+      gv[i] = gate[(size_t)(m0 + m) * ldg + (size_t)a * N + n0 + min(lane, rows - 1)];
+    }
+  }
   sp_wait_all();
   __syncthreads();
   sp_multiply<TW>(hl_smem, L);
-  const int lane = threadIdx.x & 31;
   if (lane >= rows) return;
-  for (int m = threadIdx.x >> 5; m < toks; m += SP_THREADS / 32) {
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int m = warp + i * (SP_THREADS / 32);
+    if (m >= toks) break;
     float v = sp_sum<TW>(hl_smem, L, lane, m);
-    if (gate) v *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)(m0 + m) * ldg + (size_t)a * N + n0 + lane])));
+    if (gate) v *= 1.0f / (1.0f + expf(-__bfloat162float(gv[i])));
     out[(size_t)(m0 + m) * ldo + (size_t)a * out_head + n0 + lane] = __float2bfloat16_rn(v);
   }
 }
