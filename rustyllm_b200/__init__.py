@@ -15,6 +15,7 @@ from .engine.runner import LoadInfo, Runner  # noqa: F401
 from .engine.step import Engine  # noqa: F401
 from .models import besuzen as _besuzen  # noqa: F401  (registers the architecture)
 from .models import buketar as _buketar  # noqa: F401
+from .models import tigutar as _tigutar  # noqa: F401
 from .models import forilorn as _forilorn  # noqa: F401
 from .models import llama as _llama  # noqa: F401
 from .models import mogutar as _mogutar  # noqa: F401

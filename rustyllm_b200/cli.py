@@ -286,7 +286,8 @@ def run_kernel_benchmark(runner, runs: int, as_json: bool, layer_index: int = 0)
         rows.append(("streams.join_norm", timed(lambda: blk._join(X, [(x, 1.0)], 1, blk.first_norm_request(1))),
                      (2 * blk.streams + 1) * d * 4 + d * esz))
     elif isinstance(blk.mixer_norm, LayerNorm):
-        rows.append(("attn_norm.layer", timed(lambda: K.layer_norm(x, blk.mixer_norm.weight, xn, blk.mixer_norm.eps)), d * 4))
+        rows.append(("attn_norm.layer", timed(lambda: K.layer_norm(x, blk.mixer_norm.weight, xn, blk.mixer_norm.eps, bias=blk.mixer_norm.bias)),
+                     d * 4))
     else:
         rows.append(("attn_norm.rms", timed(lambda: K.rmsnorm(x, blk.mixer_norm.weight, xn, blk.mixer_norm.eps)), d * 4))
 
@@ -360,10 +361,12 @@ def run_kernel_benchmark(runner, runs: int, as_json: bool, layer_index: int = 0)
         runner.cache.prepare([s], [1])
         q = torch.randn(1, max(qkv.shape[1], 8), device=dev).to(dt)
         o = torch.empty(1, att.H * att.vd, device=dev, dtype=dt)
-        n_qkv = (att.H + att.G) * att.hd + (0 if getattr(att, "value_from_key", False) else att.G * att.vd)
+        n_qkv = att.H * att.hd if getattr(att, "shared_keys", False) else \
+            (att.H + att.G) * att.hd + (0 if getattr(att, "value_from_key", False) else att.G * att.vd)
         gate = q[:, n_qkv:] if getattr(att, "gated", False) else None
         t = timed(lambda: K.attention(q, group.k_pool(layer), group.v_pool(layer), group.page_table, st, o, att.H, att.G, att.hd, att.scale,
-                                      att.window or 0, value_dim=att.vd, sink=getattr(att, "sink", False), gate=gate,
+                                      att.window or 0, value_dim=att.vd, sink=getattr(att, "sink", False), sinks=getattr(att, "sinks", None),
+                                      gate=gate,
                                       softcap=getattr(att, "softcap", 0.0), keep_first=getattr(att, "keep_first", 0),
                                       chunk=getattr(att, "chunk", None) or 0, gate_per_head=getattr(att, "gate_per_head", False)))
         seen = min(ctx + 1, att.window) if att.window else ctx % att.chunk + 1 if getattr(att, "chunk", None) else ctx + 1

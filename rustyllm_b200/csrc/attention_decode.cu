@@ -181,22 +181,24 @@ attention_decode_order_kernel(const int* __restrict__ seq_slots, const int* __re
   }
 }
 
-// shared memory of one CTA: the ring [warp][stage][keys | values][16 rows][HD] of bf16 (16-byte
+// shared memory of one CTA: the ring [warp][stage][keys [16][HD] | values [16][VD]] of bf16 (16-byte
 // pieces swizzled within their row), reused after the loop for the warps' (max, sum, output)
-template <int HD>
+template <int HD, int VD>
 struct DecSmem {
-  static constexpr int ROW_BYTES = HD * 2;
-  static constexpr int TILE_BYTES = DEC_BLOCK * ROW_BYTES;          // 16 keys (or values) of one KV head
-  static constexpr int STAGE_BYTES = 2 * TILE_BYTES;
+  static constexpr int ROW_BYTES = HD * 2, V_ROW_BYTES = VD * 2;
+  static constexpr int TILE_BYTES = DEC_BLOCK * ROW_BYTES;          // 16 keys of one KV head
+  static constexpr int V_TILE_BYTES = DEC_BLOCK * V_ROW_BYTES;      // 16 values
+  static constexpr int STAGE_BYTES = TILE_BYTES + V_TILE_BYTES;
   static constexpr int RING_BYTES = DEC_WARPS * DEC_STAGES * STAGE_BYTES;
-  static constexpr int MERGE_BYTES = (DEC_WARPS * 16 * (HD + 4) + 2 * DEC_WARPS * 16) * 4;
-  static constexpr int RESULT_BYTES = (16 * HD + 2 * 16) * 4;      // the CTA's own (output, max, sum), read by its cluster
+  static constexpr int MERGE_BYTES = (DEC_WARPS * 16 * (VD + 4) + 2 * DEC_WARPS * 16) * 4;
+  static constexpr int RESULT_BYTES = (16 * VD + 2 * 16) * 4;      // the CTA's own (output, max, sum), read by its cluster
   static constexpr int BYTES = RING_BYTES > MERGE_BYTES + RESULT_BYTES ? RING_BYTES : MERGE_BYTES + RESULT_BYTES;
 };
 
 // How a (sequence, head) row is finished once maximum M, denominator L and output O over all its
 // keys are known (M in the exp2 domain).  sink: the denominator has one more term of score 0 and no
-// value, p_j = e^{s_j} / (1 + sum e^{s_t}); gate: the output is multiplied by sigmoid(gate[b, h*HD + d]).
+// value, p_j = e^{s_j} / (1 + sum e^{s_t}), or with `sinks` of score sinks[h]; gate: the output is multiplied by
+// sigmoid(gate[b, h*VD + d]).
 struct DecFinish {
   int sink;
   const __nv_bfloat16* gate;
@@ -206,22 +208,25 @@ struct DecFinish {
   // in front of a window
   float softcap;
   int keep_first;
-  int gate_head;      // 0: the gate holds a number an output element; HD: one number a head (gate[b, h])
+  int gate_head;      // 0: the gate holds a number an output element; VD: one number a head (gate[b, h])
+  const float* sinks; // a score a head for the sink term, or null (score 0)
+  int value_dim;      // VD: which head an output column belongs to
 };
 
 __device__ __forceinline__ float dec_finish(float O, float L, float M, const DecFinish& f, int b, int col) {
   if (f.sink) {
-    const float M2 = fmaxf(M, 0.f);
+    const float z = f.sinks ? f.sinks[col / f.value_dim] * 1.4426950408889634f : 0.f;
+    const float M2 = fmaxf(M, z);
     const float w = exp2f(M - M2);          // exp2(-inf) = 0: a row without keys is the sink alone
     O *= w;
-    L = L * w + exp2f(-M2);
+    L = L * w + exp2f(z - M2);
   }
   float o = L > 0.f ? O / L : 0.f;
   if (f.gate) o *= 1.0f / (1.0f + expf(-__bfloat162float(f.gate[(size_t)b * f.ldg + (f.gate_head ? col / f.gate_head : col)])));
   return o;
 }
 
-template <int HD>
+template <int HD, int VD>
 __global__ void __launch_bounds__(DEC_WARPS * 32)
 attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq, const __nv_bfloat16* __restrict__ k_pool,
                         const __nv_bfloat16* __restrict__ v_pool, const int* __restrict__ page_table, int max_pages,
@@ -229,11 +234,11 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq, const __nv
                         const int4* __restrict__ plan, __nv_bfloat16* __restrict__ out, int ldo,
                         float* __restrict__ part_o, float* __restrict__ part_ml, int H, int G, float scale_log2e,
                         int window, int even_splits, DecFinish fin) {
-  constexpr int NT = HD / 8;        // output n-tiles of 8 columns
+  constexpr int NT = VD / 8;        // output n-tiles of 8 columns
   constexpr int KS = HD / 16;       // k-steps of the Q.K product
   extern __shared__ __align__(128) uint8_t dec_smem[];
-  float (*s_acc)[16][HD + 4] = reinterpret_cast<float (*)[16][HD + 4]>(dec_smem);
-  float (*s_m)[16] = reinterpret_cast<float (*)[16]>(dec_smem + DEC_WARPS * 16 * (HD + 4) * 4);
+  float (*s_acc)[16][VD + 4] = reinterpret_cast<float (*)[16][VD + 4]>(dec_smem);
+  float (*s_m)[16] = reinterpret_cast<float (*)[16]>(dec_smem + DEC_WARPS * 16 * (VD + 4) * 4);
   float (*s_l)[16] = s_m + DEC_WARPS;
 
   rl_pdl_trigger();
@@ -282,27 +287,28 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq, const __nv
   const int blk_lo = split * per_split;                                      // places
   const int blk_hi = min(blk_lo + per_split, num_blk);
   auto block_of = [&](int place) { return place < kept_blk ? place : first_blk + (place - kept_blk); };
-  const size_t page_stride = (size_t)G * RL_PAGE * HD;
-  const size_t head_off = (size_t)gkv * RL_PAGE * HD;
-
-  // A tile is 16 rows of HD bf16; the 16-byte piece `ch` of row `row` lies at
-  // row * ROW_BYTES + ((ch ^ (row & 7)) * 16).  A warp instruction copies 32 consecutive pieces.
-  constexpr int ROWB = DecSmem<HD>::ROW_BYTES, TILEB = DecSmem<HD>::TILE_BYTES, STAGEB = DecSmem<HD>::STAGE_BYTES;
-  constexpr int CH = HD / 8;                             // pieces a row
+  // A tile is 16 rows of HD (keys) or VD (values) bf16; the 16-byte piece `ch` of row `row` lies at
+  // row * row bytes + ((ch ^ (row & 7)) * 16).  A warp instruction copies 32 consecutive pieces.
+  using SM = DecSmem<HD, VD>;
+  constexpr int ROWB = SM::ROW_BYTES, TILEB = SM::TILE_BYTES, STAGEB = SM::STAGE_BYTES;
+  constexpr int VROWB = SM::V_ROW_BYTES, VTILEB = SM::V_TILE_BYTES;
   const uint32_t ring = (uint32_t)__cvta_generic_to_shared(dec_smem) + (uint32_t)(warp * DEC_STAGES * STAGEB);
   auto issue = [&](int blk, int st, int page) {
     const int key0 = blk * DEC_BLOCK;
-    const size_t base = (size_t)page * page_stride + head_off + (size_t)(key0 % RL_PAGE) * HD;
-    const __nv_bfloat16* kb = k_pool + base + 8 * lane;
-    const __nv_bfloat16* vb = v_pool + base + 8 * lane;
+    const size_t row0 = ((size_t)page * G + gkv) * RL_PAGE + key0 % RL_PAGE;
+    const size_t k_at = row0 * HD + 8 * lane, v_at = HD == VD ? k_at : row0 * VD + 8 * lane;
+    const __nv_bfloat16* kb = k_pool + k_at;
+    const __nv_bfloat16* vb = v_pool + v_at;
     const uint32_t kd = ring + (uint32_t)(st * STAGEB), vd = kd + TILEB;
 #pragma unroll
-    for (int i = 0; i < TILEB / 512; ++i) {
-      const int piece = i * 32 + lane, row = piece / CH, ch = piece % CH;
-      const uint32_t off = (uint32_t)(row * ROWB + ((ch ^ (row & 7)) << 4));
-      dec_cp_async16(kd + off, kb + i * 256, 16);
+    for (int i = 0; i < (TILEB > VTILEB ? TILEB : VTILEB) / 512; ++i) {
+      const int piece = i * 32 + lane;
+      const int k_r = piece / (HD / 8), v_r = piece / (VD / 8);
+      const uint32_t k_off = (uint32_t)(k_r * ROWB + (((piece % (HD / 8)) ^ (k_r & 7)) << 4));
+      const uint32_t v_off = (uint32_t)(v_r * VROWB + (((piece % (VD / 8)) ^ (v_r & 7)) << 4));
+      if (i < TILEB / 512) dec_cp_async16(kd + k_off, kb + i * 256, 16);
       // rows beyond the sequence may hold anything: zeros instead (their weights are zero)
-      dec_cp_async16(vd + off, vb + i * 256, key0 + row < len ? 16 : 0);
+      if (i < VTILEB / 512) dec_cp_async16(vd + v_off, vb + i * 256, key0 + v_r < len ? 16 : 0);
     }
   };
   // ldmatrix row addresses of this lane within a tile.  Keys (as they lie): matrix lane/8 is piece
@@ -310,7 +316,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq, const __nv
   // of keys (lane & 7) + 8 * ((lane / 8) & 1).
   const int swz = lane & 7;
   const uint32_t k_row = (uint32_t)(swz * ROWB), k_piece = (uint32_t)(lane >> 3);
-  const uint32_t v_row = (uint32_t)((swz + 8 * ((lane >> 3) & 1)) * ROWB), v_piece = (uint32_t)(lane >> 4);
+  const uint32_t v_row = (uint32_t)((swz + 8 * ((lane >> 3) & 1)) * VROWB), v_piece = (uint32_t)(lane >> 4);
 
   {
     int first_pages[DEC_STAGES - 1];
@@ -428,8 +434,8 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq, const __nv
     if (g + 8 < m) *reinterpret_cast<float2*>(&s_acc[warp][g + 8][d0]) = make_float2(acc[j][2], acc[j][3]);
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < m * HD; idx += DEC_WARPS * 32) {
-    const int r = idx / HD, d = idx % HD;
+  for (int idx = threadIdx.x; idx < m * VD; idx += DEC_WARPS * 32) {
+    const int r = idx / VD, d = idx % VD;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < DEC_WARPS; ++w) M = fmaxf(M, s_m[w][r]);
@@ -442,42 +448,42 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq, const __nv
     }
     const int h = gkv * m + r;
     if (direct) {
-      out[(size_t)b * ldo + (size_t)h * HD + d] = __float2bfloat16_rn(dec_finish(O, L, M, fin, b, h * HD + d));
+      out[(size_t)b * ldo + (size_t)h * VD + d] = __float2bfloat16_rn(dec_finish(O, L, M, fin, b, h * VD + d));
     } else if (clustered) {
-      float* c_o = reinterpret_cast<float*>(dec_smem + DecSmem<HD>::MERGE_BYTES);
-      c_o[r * HD + d] = O;
-      if (d == 0) { c_o[16 * HD + r] = M; c_o[16 * HD + 16 + r] = L; }
+      float* c_o = reinterpret_cast<float*>(dec_smem + SM::MERGE_BYTES);
+      c_o[r * VD + d] = O;
+      if (d == 0) { c_o[16 * VD + r] = M; c_o[16 * VD + 16 + r] = L; }
     } else {
       const size_t p = (size_t)chunk_id * H + h;           // partial results lie in the order of the chunks
-      part_o[p * HD + d] = O;
+      part_o[p * VD + d] = O;
       if (d == 0) { part_ml[2 * p] = M; part_ml[2 * p + 1] = L; }
     }
   }
   if (clustered) {
     // every chunk of the sequence has its result in shared memory; this CTA finishes its share
-    // of the m x HD outputs, adding the chunks in their order
+    // of the m x VD outputs, adding the chunks in their order
     dec_cluster_sync();
-    const float* c_o = reinterpret_cast<const float*>(dec_smem + DecSmem<HD>::MERGE_BYTES);
-    const int per = (m * HD + num_splits - 1) / num_splits;
-    const int lo = split * per, hi = min(lo + per, m * HD);
+    const float* c_o = reinterpret_cast<const float*>(dec_smem + SM::MERGE_BYTES);
+    const int per = (m * VD + num_splits - 1) / num_splits;
+    const int lo = split * per, hi = min(lo + per, m * VD);
     for (int idx = lo + threadIdx.x; idx < hi; idx += DEC_WARPS * 32) {
-      const int r = idx / HD, d = idx % HD;
+      const int r = idx / VD, d = idx % VD;
       float M = -INFINITY;
-      for (int c = 0; c < num_splits; ++c) M = fmaxf(M, dec_peer_f32(c_o + 16 * HD + r, c));
+      for (int c = 0; c < num_splits; ++c) M = fmaxf(M, dec_peer_f32(c_o + 16 * VD + r, c));
       float L = 0.f, O = 0.f;
       for (int c = 0; c < num_splits; ++c) {
-        const float mc = dec_peer_f32(c_o + 16 * HD + r, c);
+        const float mc = dec_peer_f32(c_o + 16 * VD + r, c);
         const float wgt = (mc > -INFINITY) ? exp2f(mc - M) : 0.f;
-        L += dec_peer_f32(c_o + 16 * HD + 16 + r, c) * wgt;
-        O += dec_peer_f32(c_o + r * HD + d, c) * wgt;
+        L += dec_peer_f32(c_o + 16 * VD + 16 + r, c) * wgt;
+        O += dec_peer_f32(c_o + r * VD + d, c) * wgt;
       }
-      out[(size_t)b * ldo + (size_t)(gkv * m + r) * HD + d] = __float2bfloat16_rn(dec_finish(O, L, M, fin, b, (gkv * m + r) * HD + d));
+      out[(size_t)b * ldo + (size_t)(gkv * m + r) * VD + d] = __float2bfloat16_rn(dec_finish(O, L, M, fin, b, (gkv * m + r) * VD + d));
     }
     dec_cluster_sync();      // nobody leaves while its shared memory may still be read
   }
 }
 
-// Combines the chunks of one (sequence, head) in chunk order.
+// Combines the chunks of one (sequence, head) in chunk order.  HD: the width of a value head.
 template <int HD>
 __global__ void attention_decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                 const int2* __restrict__ plan_seqs, int even_splits,
@@ -532,15 +538,15 @@ __global__ void attention_decode_combine_kernel(const float* __restrict__ part_o
   }
 }
 
-template <int HD>
+template <int HD, int VD>
 static int launch_decode(const void* q, int ldq, const void* k_pool, const void* v_pool, const int* page_table,
                          int max_pages, const int* seq_slots, const int* kv_lens, void* out, int ldo,
                          float* part_o, float* part_ml, const int* plan, int B, int H, int G, float scale, int window,
                          int num_splits, DecFinish fin, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, DecSmem<HD>::BYTES);
-    RL_REQUIRE(e == cudaSuccess, "rl_attention_decode: cannot reserve %d bytes of shared memory: %s", DecSmem<HD>::BYTES, cudaGetErrorString(e));
+    cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<HD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, DecSmem<HD, VD>::BYTES);
+    RL_REQUIRE(e == cudaSuccess, "rl_attention_decode: cannot reserve %d bytes of shared memory: %s", DecSmem<HD, VD>::BYTES, cudaGetErrorString(e));
     configured = true;
   }
   const int nchunk = B * num_splits;
@@ -552,7 +558,7 @@ static int launch_decode(const void* q, int ldq, const void* k_pool, const void*
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;
     cfg.blockDim = dim3(DEC_WARPS * 32);
-    cfg.dynamicSmemBytes = DecSmem<HD>::BYTES;
+    cfg.dynamicSmemBytes = DecSmem<HD, VD>::BYTES;
     cfg.stream = stream;
     cudaLaunchAttribute attr[2];
     int na = 0;
@@ -566,7 +572,7 @@ static int launch_decode(const void* q, int ldq, const void* k_pool, const void*
     ++na;
     cfg.attrs = attr;
     cfg.numAttrs = na;
-    cudaError_t e = cudaLaunchKernelEx(&cfg, attention_decode_kernel<HD>,
+    cudaError_t e = cudaLaunchKernelEx(&cfg, attention_decode_kernel<HD, VD>,
         (const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, page_table, max_pages,
         seq_slots, kv_lens, (const int4*)nullptr, (__nv_bfloat16*)out, ldo, (float*)nullptr, (float*)nullptr, H, G,
         scale * 1.4426950408889634f, window, num_splits, fin);
@@ -575,25 +581,28 @@ static int launch_decode(const void* q, int ldq, const void* k_pool, const void*
     return RL_OK;
   }
   dim3 grid(G, nchunk);
-  rl_launch_pdl(attention_decode_kernel<HD>, grid, dim3(DEC_WARPS * 32), (size_t)DecSmem<HD>::BYTES, stream,
+  rl_launch_pdl(attention_decode_kernel<HD, VD>, grid, dim3(DEC_WARPS * 32), (size_t)DecSmem<HD, VD>::BYTES, stream,
       (const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, page_table, max_pages,
       seq_slots, kv_lens, entries, (__nv_bfloat16*)out, ldo, part_o, part_ml, H, G, scale * 1.4426950408889634f, window,
       num_splits, fin);
   RL_LAUNCH_CHECK("rl_attention_decode");
   if (num_splits > 1) {
-    rl_launch_pdl(attention_decode_combine_kernel<HD>, dim3(H, B), dim3(HD), 0, stream,
+    rl_launch_pdl(attention_decode_combine_kernel<VD>, dim3(H, B), dim3(VD), 0, stream,
                   (const float*)part_o, (const float*)part_ml, seqs, num_splits, (__nv_bfloat16*)out, ldo, H, fin);
     RL_LAUNCH_CHECK("rl_attention_decode (combine)");
   }
   return RL_OK;
 }
 
-// 1 if the decode kernel takes this shape: bf16, head_dim 64 or 128, at most 16 query
+// 1 if the decode kernel takes this shape: bf16, key and value heads of 64 or 128, at most 16 query
 // heads per KV head.  Other shapes go to the any-shape kernel.
-extern "C" int rl_attention_decode_supported(int num_heads, int num_kv_heads, int head_dim) {
+extern "C" int rl_attention_decode_supported_shaped(int num_heads, int num_kv_heads, int head_dim, int value_dim) {
   if (num_kv_heads <= 0 || num_heads % num_kv_heads != 0) return 0;
   if (num_heads / num_kv_heads > 16) return 0;
-  return head_dim == 64 || head_dim == 128;
+  return (head_dim == 64 || head_dim == 128) && (value_dim == 64 || value_dim == 128);
+}
+extern "C" int rl_attention_decode_supported(int num_heads, int num_kv_heads, int head_dim) {
+  return rl_attention_decode_supported_shaped(num_heads, num_kv_heads, head_dim, head_dim);
 }
 
 // Ints of a plan for the given sizes (0 with one split): 4 a chunk, 2 a sequence.
@@ -629,26 +638,29 @@ extern "C" int rl_attention_decode_plan(const int* seq_slots, const int* kv_lens
 // How many CTAs of the decode kernel the GPU holds at once at this head size (CTAs an SM by shared
 // memory and registers, times SMs), and how many bytes of keys and values one CTA keeps in flight:
 // what the choice between equal chunks, whole sequences and dealt chunks goes by.
-extern "C" int rl_attention_decode_places(int head_dim) {
-  static int places[2] = {0, 0};
-  RL_REQUIRE(head_dim == 64 || head_dim == 128, "rl_attention_decode_places: head_dim %d is not 64 or 128", head_dim);
-  int& p = places[head_dim == 128];
+template <int HD, int VD>
+static int decode_places() {
+  static int p = 0;
   if (p == 0) {
     int per_sm = 0;
-    cudaError_t e;
-    if (head_dim == 64) {
-      e = cudaFuncSetAttribute(attention_decode_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, DecSmem<64>::BYTES);
-      if (e == cudaSuccess) e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, attention_decode_kernel<64>, DEC_WARPS * 32, DecSmem<64>::BYTES);
-    } else {
-      e = cudaFuncSetAttribute(attention_decode_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, DecSmem<128>::BYTES);
-      if (e == cudaSuccess) e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, attention_decode_kernel<128>, DEC_WARPS * 32, DecSmem<128>::BYTES);
-    }
+    cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<HD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, DecSmem<HD, VD>::BYTES);
+    if (e == cudaSuccess) e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, attention_decode_kernel<HD, VD>, DEC_WARPS * 32, DecSmem<HD, VD>::BYTES);
     RL_REQUIRE(e == cudaSuccess && per_sm > 0, "rl_attention_decode_places: occupancy query failed: %s", cudaGetErrorString(e));
     p = per_sm * rl_num_sms();
   }
   return p;
 }
-extern "C" int rl_attention_decode_ring_bytes(int head_dim) { return head_dim == 64 ? DecSmem<64>::RING_BYTES : DecSmem<128>::RING_BYTES; }
+extern "C" int rl_attention_decode_places_shaped(int head_dim, int value_dim) {
+  RL_REQUIRE((head_dim == 64 || head_dim == 128) && (value_dim == 64 || value_dim == 128),
+             "rl_attention_decode_places: heads of %d and values of %d are not 64 or 128", head_dim, value_dim);
+  if (head_dim == 64) return value_dim == 64 ? decode_places<64, 64>() : decode_places<64, 128>();
+  return value_dim == 64 ? decode_places<128, 64>() : decode_places<128, 128>();
+}
+extern "C" int rl_attention_decode_places(int head_dim) { return rl_attention_decode_places_shaped(head_dim, head_dim); }
+extern "C" int rl_attention_decode_ring_bytes_shaped(int head_dim, int value_dim) {
+  return DEC_WARPS * DEC_STAGES * DEC_BLOCK * (head_dim + value_dim) * 2;
+}
+extern "C" int rl_attention_decode_ring_bytes(int head_dim) { return rl_attention_decode_ring_bytes_shaped(head_dim, head_dim); }
 
 // Ints of an order plan for num_seqs sequences.
 extern "C" long long rl_attention_decode_order_ints(int num_seqs) { return 6LL * num_seqs; }
@@ -683,22 +695,26 @@ extern "C" int rl_attention_decode_order(const int* seq_slots, const int* kv_len
 // softcap * tanh(s / softcap).  keep_first > 0 (with a window): positions [0, keep_first) stay visible.
 // window < 0: a chunked mask with blocks of -window positions (the query sees its own block up to itself).
 // gate_per_head != 0: the gate is [num_seqs, ldg] with one number a head, sigmoid(gate[b, h]) on all of head h's output.
-extern "C" int rl_attention_decode_headgate(const void* q, int ldq, const void* k_pool, const void* v_pool,
+//
+// rl_attention_decode_wide: value heads of their own width (value_dim; out is [B, ldo] with head h at h * value_dim, the
+// scratch counts value_dim floats a partial result), and sinks (float [num_heads], may be null): with sink != 0 the extra
+// term has the score sinks[h] instead of 0 (no scale, no soft cap).
+extern "C" int rl_attention_decode_wide(const void* q, int ldq, const void* k_pool, const void* v_pool,
                                             const int* page_table, int max_pages, const int* seq_slots, const int* kv_lens,
                                             void* out, int ldo, float* scratch, const int* plan, int num_seqs, int num_heads,
                                             int num_kv_heads, int head_dim, float scale, int window, int num_splits,
                                             int sink, const void* gate, int ldg, float softcap, int keep_first, int gate_per_head,
-                                            cudaStream_t stream) {
-  RL_REQUIRE(gate == nullptr || ldg >= (gate_per_head ? num_heads : num_heads * head_dim), "rl_attention_decode: the gate's row stride is too small");
+                                            int value_dim, const float* sinks, cudaStream_t stream) {
+  RL_REQUIRE(gate == nullptr || ldg >= (gate_per_head ? num_heads : num_heads * value_dim), "rl_attention_decode: the gate's row stride is too small");
   RL_REQUIRE(softcap >= 0.f && keep_first >= 0, "rl_attention_decode: negative soft cap or number of kept first tokens");
-  const DecFinish fin = {sink, (const __nv_bfloat16*)gate, ldg, softcap, window > 0 ? keep_first : 0, gate_per_head ? head_dim : 0};
-  RL_REQUIRE(rl_attention_decode_supported(num_heads, num_kv_heads, head_dim),
-             "rl_attention_decode: unsupported shape (heads %d, KV heads %d, head_dim %d): needs head_dim 64 or 128 "
-             "and at most 16 heads per KV head", num_heads, num_kv_heads, head_dim);
+  const DecFinish fin = {sink, (const __nv_bfloat16*)gate, ldg, softcap, window > 0 ? keep_first : 0, gate_per_head ? value_dim : 0, sinks, value_dim};
+  RL_REQUIRE(rl_attention_decode_supported_shaped(num_heads, num_kv_heads, head_dim, value_dim),
+             "rl_attention_decode: unsupported shape (heads %d, KV heads %d, head_dim %d, value_dim %d): needs heads of 64 or 128 "
+             "and at most 16 heads per KV head", num_heads, num_kv_heads, head_dim, value_dim);
   RL_REQUIRE(num_seqs >= 0 && num_splits >= 1, "rl_attention_decode: bad sizes");
   RL_REQUIRE(num_seqs <= 65535 && num_kv_heads <= 65535 && (long long)num_seqs * num_splits <= 65535,
              "rl_attention_decode: too many sequences, chunks (%d x %d splits) or KV heads for one grid", num_seqs, num_splits);
-  RL_REQUIRE(ldq >= num_heads * head_dim && ldo >= num_heads * head_dim && ldq % 8 == 0,
+  RL_REQUIRE(ldq >= num_heads * head_dim && ldo >= num_heads * value_dim && ldq % 8 == 0,
              "rl_attention_decode: row strides too small or not a multiple of 8 elements");
   RL_REQUIRE(((uintptr_t)q & 15) == 0 && ((uintptr_t)k_pool & 15) == 0 && ((uintptr_t)v_pool & 15) == 0,
              "rl_attention_decode: q and the cache pools must be 16-byte aligned");
@@ -708,12 +724,24 @@ extern "C" int rl_attention_decode_headgate(const void* q, int ldq, const void* 
   if (num_seqs == 0) return RL_OK;
   const size_t parts = (size_t)num_seqs * num_heads * num_splits;
   float* part_o = scratch;
-  float* part_ml = scratch ? scratch + parts * head_dim : nullptr;
-  if (head_dim == 64)
-    return launch_decode<64>(q, ldq, k_pool, v_pool, page_table, max_pages, seq_slots, kv_lens, out, ldo, part_o,
-                             part_ml, plan, num_seqs, num_heads, num_kv_heads, scale, window, num_splits, fin, stream);
-  return launch_decode<128>(q, ldq, k_pool, v_pool, page_table, max_pages, seq_slots, kv_lens, out, ldo, part_o,
-                            part_ml, plan, num_seqs, num_heads, num_kv_heads, scale, window, num_splits, fin, stream);
+  float* part_ml = scratch ? scratch + parts * value_dim : nullptr;
+#define DEC_GO(HD, VD)                                                                                                    \
+  launch_decode<HD, VD>(q, ldq, k_pool, v_pool, page_table, max_pages, seq_slots, kv_lens, out, ldo, part_o, part_ml,     \
+                        plan, num_seqs, num_heads, num_kv_heads, scale, window, num_splits, fin, stream)
+  if (head_dim == 64) return value_dim == 64 ? DEC_GO(64, 64) : DEC_GO(64, 128);
+  return value_dim == 64 ? DEC_GO(128, 64) : DEC_GO(128, 128);
+#undef DEC_GO
+}
+
+extern "C" int rl_attention_decode_headgate(const void* q, int ldq, const void* k_pool, const void* v_pool,
+                                            const int* page_table, int max_pages, const int* seq_slots, const int* kv_lens,
+                                            void* out, int ldo, float* scratch, const int* plan, int num_seqs, int num_heads,
+                                            int num_kv_heads, int head_dim, float scale, int window, int num_splits,
+                                            int sink, const void* gate, int ldg, float softcap, int keep_first, int gate_per_head,
+                                            cudaStream_t stream) {
+  return rl_attention_decode_wide(q, ldq, k_pool, v_pool, page_table, max_pages, seq_slots, kv_lens, out, ldo, scratch, plan,
+                                  num_seqs, num_heads, num_kv_heads, head_dim, scale, window, num_splits, sink, gate, ldg, softcap,
+                                  keep_first, gate_per_head, head_dim, nullptr, stream);
 }
 
 extern "C" int rl_attention_decode_masked(const void* q, int ldq, const void* k_pool, const void* v_pool,

@@ -54,18 +54,19 @@ constexpr int FA_PV_WARP = 2;
 constexpr int FA_REGS_FEED = 56, FA_REGS_SOFTMAX = 224;
 constexpr uint32_t FA_WAIT_LIMIT = 1u << 22;
 constexpr int HALF_BYTES = 128 * 64 * 2;               // [128 rows x 64 bf16], 16 KB
-// sizes that depend on the head size HD (64 or 128): a head is HD / 64 halves of 64 dimensions
-template <int HD> struct FaSizes {
-  static constexpr int HALVES = HD / 64;
+// sizes that depend on the widths of a key head HD and of a value head VD (64 or 128 each): halves of 64 dimensions
+template <int HD, int VD> struct FaSizes {
+  static constexpr int HALVES = HD / 64, V_HALVES = VD / 64;
   static constexpr int Q_BYTES = HALVES * HALF_BYTES;          // 16 or 32 KB
-  static constexpr int TILE_BYTES = HALVES * HALF_BYTES;       // a key tile or a value tile: 16 or 32 KB
+  static constexpr int TILE_BYTES = HALVES * HALF_BYTES;       // a key tile: 16 or 32 KB
+  static constexpr int V_TILE_BYTES = V_HALVES * HALF_BYTES;   // a value tile
   // keys are asked for a tile further ahead than values: the scores of a tile are computed as soon as the
   // buffer is free, a whole tile before its P V
   static constexpr int K_STAGES = HD == 64 ? 4 : 3;
-  static constexpr int V_STAGES = HD == 64 ? 3 : 2;
+  static constexpr int V_STAGES = VD == 64 ? 3 : 2;
   // + alignment slack, barriers, and the softmax threads' exchange: running maxima (two tiles in turn), and the
   // groups' last maxima and sums
-  static constexpr int SMEM = Q_BYTES + (K_STAGES + V_STAGES) * TILE_BYTES + 1024 + 512 + 3 * 2 * TQ * 4;
+  static constexpr int SMEM = Q_BYTES + K_STAGES * TILE_BYTES + V_STAGES * V_TILE_BYTES + 1024 + 512 + 3 * 2 * TQ * 4;
 };
 constexpr float LAZY_LOG2 = 8.0f;                      // rescale O only when the maximum grew by more than 2^8
 
@@ -188,7 +189,7 @@ __host__ __device__ constexpr uint32_t fa_idesc(int m, int n, int b_mn) {
   return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)b_mn << 16) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
 }
 
-template <int HD>
+template <int HD, int VD>
 __global__ void __launch_bounds__(FA_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const int* __restrict__ page_table, int max_pages,
@@ -196,15 +197,16 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ kv_lens, int num_seqs, __nv_bfloat16* __restrict__ out, int ldo,
                             int H, int G, float scale_log2e, int window, int* __restrict__ err,
                             const int* __restrict__ tile_order, int sink, const __nv_bfloat16* __restrict__ gate, int ldg,
-                            float cap_in, float cap_out, int keep_first, int chunk, int gate_per_head) {
+                            float cap_in, float cap_out, int keep_first, int chunk, int gate_per_head, const float* __restrict__ sinks) {
   extern __shared__ uint8_t fa_smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)fa_smem_raw + 1023) & ~(uintptr_t)1023);
   uint8_t* q_tile = smem;                                   // [2 halves][128 x 64]
-  constexpr int HALVES = FaSizes<HD>::HALVES, Q_BYTES = FaSizes<HD>::Q_BYTES, TILE_BYTES = FaSizes<HD>::TILE_BYTES;
-  constexpr int K_STAGES = FaSizes<HD>::K_STAGES, V_STAGES = FaSizes<HD>::V_STAGES;
+  using SZ = FaSizes<HD, VD>;
+  constexpr int HALVES = SZ::HALVES, V_HALVES = SZ::V_HALVES, Q_BYTES = SZ::Q_BYTES, TILE_BYTES = SZ::TILE_BYTES, V_TILE_BYTES = SZ::V_TILE_BYTES;
+  constexpr int K_STAGES = SZ::K_STAGES, V_STAGES = SZ::V_STAGES;
   uint8_t* k_ring = smem + Q_BYTES;                         // [stage][halves]
   uint8_t* v_ring = k_ring + K_STAGES * TILE_BYTES;         // [stage][halves]
-  uint64_t* bars = (uint64_t*)(v_ring + V_STAGES * TILE_BYTES);
+  uint64_t* bars = (uint64_t*)(v_ring + V_STAGES * V_TILE_BYTES);
   uint64_t* q_full = bars;                 // 1
   uint64_t* k_full = bars + 1;             // keys and values have rings of their own
   uint64_t* k_empty = k_full + K_STAGES;
@@ -271,7 +273,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   fa_fence_after();
   const uint32_t tmem_base = *tmem_slot;
   // S buffers at columns 0 and 128, O at 256, the two P buffers (64 columns each) behind O
-  const uint32_t tmem_s0 = tmem_base, tmem_o = tmem_base + 256, tmem_p = tmem_base + 256 + HD;
+  const uint32_t tmem_s0 = tmem_base, tmem_o = tmem_base + 256, tmem_p = tmem_base + 256 + VD;
   const int b = *s_seq;
   const bool have_work = b < num_seqs;      // the grid is sized exactly; defensive
   const int h = blockIdx.x, gkv = h / (H / G);
@@ -312,11 +314,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           const int p1 = (2 * kt + 1) * RL_PAGE < kv_len ? pages[2 * kt + 1] : p0;   // beyond the sequence: any valid page (all masked)
           const int r0 = (p0 * G + gkv) * RL_PAGE, r1 = (p1 * G + gkv) * RL_PAGE;
           const uint32_t fb = fa_smem_u32(values ? &v_full[st] : &k_full[st]);
-          uint8_t* base = (values ? v_ring : k_ring) + (size_t)st * TILE_BYTES;
+          uint8_t* base = values ? v_ring + (size_t)st * V_TILE_BYTES : k_ring + (size_t)st * TILE_BYTES;
           const CUtensorMap* map = values ? &map_v : &map_k;
-          fa_expect_tx(fb, TILE_BYTES);
-#pragma unroll
-          for (int half = 0; half < HALVES; ++half) {     // 64 head dimensions a half; 64 positions a page
+          fa_expect_tx(fb, values ? V_TILE_BYTES : TILE_BYTES);
+          for (int half = 0; half < (values ? V_HALVES : HALVES); ++half) {     // 64 head dimensions a half; 64 positions a page
             fa_tma_2d(fa_smem_u32(base + half * HALF_BYTES), map, fb, 64 * half, r0);
             fa_tma_2d(fa_smem_u32(base + half * HALF_BYTES + 64 * 128), map, fb, 64 * half, r1);
           }
@@ -372,13 +373,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     } else if (warp == FA_PV_WARP) {
       if (lane == 0 && have_work) {
         // ---------------- issuer of O += P V ----------------
-        constexpr uint32_t idesc_o = fa_idesc(TQ, HD, 1);     // P in tensor memory, V MN-major
+        constexpr uint32_t idesc_o = fa_idesc(TQ, VD, 1);     // P in tensor memory, V MN-major
         bool ok = true;
         for (int i = 0; i < num_kt && ok; ++i) {
           if (!fa_wait(fa_smem_u32(&v_full[i % V_STAGES]), (i / V_STAGES) & 1, abort_flag)) { ok = false; break; }
           if (!fa_wait(fa_smem_u32(&p_full[i & 1]), (i >> 1) & 1, abort_flag)) { ok = false; break; }
           fa_fence_after();
-          uint8_t* vbase = v_ring + (size_t)(i % V_STAGES) * TILE_BYTES;
+          uint8_t* vbase = v_ring + (size_t)(i % V_STAGES) * V_TILE_BYTES;
 #pragma unroll
           for (int k = 0; k < TK / 16; ++k) {                 // 16 positions a step
             // P of this tile: 16 keys = 8 columns of packed bf16 pairs a step, in the P buffer of its parity
@@ -396,7 +397,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(FA_REGS_SOFTMAX));
     if (have_work) {
       // ---------------- softmax warps: group 0 takes the even key tiles, group 1 the odd ones ----------------
-      constexpr int OC = HD / 2;                              // output columns a thread writes at the end
+      constexpr int OC = VD / 2;                              // output columns a thread writes at the end
       const int quarter = warp & 3, grp = (warp - 4) >> 2;
       const int r = quarter * 32 + lane;                      // row of the tile = lane of tensor memory
       const int pos = start_pos + qt0 + r;                    // position of this row's query
@@ -529,7 +530,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           if (!ok) break;
           fa_fence_after();
 #pragma unroll 1
-          for (int c = 0; c < HD / 32; ++c) {               // the whole row of O
+          for (int c = 0; c < VD / 32; ++c) {               // the whole row of O
             uint32_t v[32];
             const uint32_t o_addr = tmem_o + lane_addr + (uint32_t)(c * 32);
             fa_ld32(o_addr, v);
@@ -567,12 +568,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const float w_mine = m_mine == -INFINITY ? 0.f : fa_exp2(m_mine - m_fin);
         const float w_other = m_other == -INFINITY ? 0.f : fa_exp2(m_other - m_fin);
         const float l_row = grp == 0 ? l_run * w_mine + l_other * w_other : l_other * w_other + l_run * w_mine;
-        // sink: one more term in the denominator, of score 0 and without a value; O and the sums are in
-        // units of exp2(-m_fin), so the term is exp2(0 - m_fin) (a row without keys: 1 / inf = 0)
-        const float l_all = sink ? l_row + fa_exp2(-m_fin) : l_row;
+        // sink: one more term in the denominator, without a value, of score 0 or the head's own (sinks[h]); O and the
+        // sums are in units of exp2(-m_fin), so the term is exp2(score - m_fin) (a row without keys: 1 / inf = 0)
+        const float sink_score = sinks ? sinks[h] * 1.4426950408889634f : 0.f;
+        const float l_all = sink ? l_row + fa_exp2(sink_score - m_fin) : l_row;
         float inv = l_all > 0.f ? 1.0f / l_all : 0.f;
-        __nv_bfloat16* orow = out + (size_t)(row0 + qt0 + r) * ldo + (size_t)h * HD + grp * OC;
-        const __nv_bfloat16* grow = (gate && !gate_per_head) ? gate + (size_t)(row0 + qt0 + r) * ldg + (size_t)h * HD + grp * OC : nullptr;
+        __nv_bfloat16* orow = out + (size_t)(row0 + qt0 + r) * ldo + (size_t)h * VD + grp * OC;
+        const __nv_bfloat16* grow = (gate && !gate_per_head) ? gate + (size_t)(row0 + qt0 + r) * ldg + (size_t)h * VD + grp * OC : nullptr;
         if (gate && gate_per_head && r < rows_here)      // one number a head: sigmoid(gate[m, h]) on the whole row, in 32-bit
           inv *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)(row0 + qt0 + r) * ldg + h])));
 #pragma unroll 1
@@ -641,12 +643,31 @@ int fa_make_map(CUtensorMap* map, const void* base, long long rows, int cols, lo
   return RL_OK;
 }
 
+template <int HD, int VD, typename... Args>
+int fa_launch(dim3 grid, cudaStream_t stream, Args... args) {
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, FaSizes<HD, VD>::SMEM);
+    RL_REQUIRE(e == cudaSuccess, "rl_attention_prefill_tc: cannot reserve %d bytes of shared memory: %s", FaSizes<HD, VD>::SMEM, cudaGetErrorString(e));
+    configured = true;
+  }
+  cudaError_t e = rl_launch_pdl(attention_prefill_tc_kernel<HD, VD>, grid, dim3(FA_THREADS), (size_t)FaSizes<HD, VD>::SMEM, stream, args...);
+  if (e != cudaSuccess) {
+    rl_set_error("rl_attention_prefill_tc: launch failed: %s", cudaGetErrorString(e));
+    return RL_ERR_CUDA;
+  }
+  return RL_OK;
+}
+
 }  // namespace
 
-// 1 if the tcgen05 prefill kernel takes this shape: head size 64 or 128.
-extern "C" int rl_attention_prefill_tc_supported(int num_heads, int num_kv_heads, int head_dim) {
+// 1 if the tcgen05 prefill kernel takes this shape: key and value heads of 64 or 128.
+extern "C" int rl_attention_prefill_tc_supported_shaped(int num_heads, int num_kv_heads, int head_dim, int value_dim) {
   if (num_kv_heads <= 0 || num_heads % num_kv_heads != 0) return 0;
-  return head_dim == 64 || head_dim == 128;
+  return (head_dim == 64 || head_dim == 128) && (value_dim == 64 || value_dim == 128);
+}
+extern "C" int rl_attention_prefill_tc_supported(int num_heads, int num_kv_heads, int head_dim) {
+  return rl_attention_prefill_tc_supported_shaped(num_heads, num_kv_heads, head_dim, head_dim);
 }
 
 // Same interface as rl_attention_prefill, with num_tiles = sum over sequences of
@@ -662,6 +683,49 @@ extern "C" int rl_attention_prefill_tc_supported(int num_heads, int num_kv_heads
 // positions [p - p % chunk, p], the positions of its own block counted from the sequence's start.
 // gate_per_head != 0: the gate is bf16 [M, ldg] with one number a head (no alignment rule): sigmoid(gate[m, h]) on all of
 // head h's output.
+//
+// rl_attention_prefill_tc_wide: value heads of their own width (value_dim; out holds head h at h * value_dim), and sinks
+// (float [num_heads], may be null): with sink != 0 the extra term has the score sinks[h] instead of 0.
+extern "C" int rl_attention_prefill_tc_wide(const void* q, int ldq, const void* k_pool, const void* v_pool, int num_pages,
+                                                const int* page_table, int max_pages, const int* cu_seqlens,
+                                                const int* seq_slots, const int* kv_lens, int num_seqs, int num_tiles,
+                                                int num_tokens, void* out, int ldo, int num_heads, int num_kv_heads, int head_dim,
+                                                float scale, int window, int* err, const int* tile_order, int sink,
+                                                const void* gate, int ldg, float softcap, int keep_first, int chunk, int gate_per_head,
+                                                int value_dim, const float* sinks, cudaStream_t stream) {
+  RL_REQUIRE(chunk >= 0 && !(chunk > 0 && window > 0), "rl_attention_prefill_tc: a chunked mask and a window exclude one another");
+  RL_REQUIRE(softcap >= 0.f && keep_first >= 0 && scale > 0.f, "rl_attention_prefill_tc: negative soft cap or number of kept first tokens, or a scale that is not positive");
+  const float cap_in = softcap > 0.f ? scale / softcap : 0.f, cap_out = softcap > 0.f ? softcap / scale : 0.f;
+  if (window <= 0) keep_first = 0;
+  RL_REQUIRE(gate == nullptr || (gate_per_head && ldg >= num_heads) || (!gate_per_head && ldg >= num_heads * value_dim && ldg % 8 == 0 && ((uintptr_t)gate & 15) == 0),
+             "rl_attention_prefill_tc: the gate must be 16-byte aligned with a row stride that is a multiple of 8 and holds all heads");
+  RL_REQUIRE(rl_attention_prefill_tc_supported_shaped(num_heads, num_kv_heads, head_dim, value_dim),
+             "rl_attention_prefill_tc: unsupported shape (heads %d, KV heads %d, head_dim %d, value_dim %d): needs heads of 64 or 128",
+             num_heads, num_kv_heads, head_dim, value_dim);
+  RL_REQUIRE(num_seqs >= 0 && num_tiles >= 0 && num_tokens >= 0 && num_pages > 0 && num_tiles <= 65535, "rl_attention_prefill_tc: bad sizes");
+  RL_REQUIRE(ldq >= num_heads * head_dim && ldq % 8 == 0 && ldo >= num_heads * value_dim && ldo % 8 == 0,
+             "rl_attention_prefill_tc: row strides must be multiples of 8 elements and hold all heads");
+  RL_REQUIRE(((uintptr_t)q & 15) == 0 && ((uintptr_t)out & 15) == 0 && ((uintptr_t)k_pool & 15) == 0 && ((uintptr_t)v_pool & 15) == 0,
+             "rl_attention_prefill_tc: pointers must be 16-byte aligned");
+  RL_REQUIRE(window >= 0 && err != nullptr, "rl_attention_prefill_tc: negative window or null error word");
+  if (num_seqs == 0 || num_tiles == 0) return RL_OK;
+  CUtensorMap mq, mk, mv;
+  int rc = fa_make_map(&mq, q, num_tokens, num_heads * head_dim, ldq, TQ);
+  if (rc != RL_OK) return rc;
+  const long long pool_rows = (long long)num_pages * num_kv_heads * RL_PAGE;
+  rc = fa_make_map(&mk, k_pool, pool_rows, head_dim, head_dim, RL_PAGE);
+  if (rc != RL_OK) return rc;
+  rc = fa_make_map(&mv, v_pool, pool_rows, value_dim, value_dim, RL_PAGE);
+  if (rc != RL_OK) return rc;
+#define FA_GO(HD, VD)                                                                                                          \
+  fa_launch<HD, VD>(dim3(num_heads, num_tiles), stream, mq, mk, mv, page_table, max_pages, cu_seqlens, seq_slots, kv_lens,     \
+                    num_seqs, (__nv_bfloat16*)out, ldo, num_heads, num_kv_heads, scale * 1.4426950408889634f, window, err,      \
+                    tile_order, sink, (const __nv_bfloat16*)gate, ldg, cap_in, cap_out, keep_first, chunk, gate_per_head, sinks)
+  if (head_dim == 64) return value_dim == 64 ? FA_GO(64, 64) : FA_GO(64, 128);
+  return value_dim == 64 ? FA_GO(128, 64) : FA_GO(128, 128);
+#undef FA_GO
+}
+
 extern "C" int rl_attention_prefill_tc_headgate(const void* q, int ldq, const void* k_pool, const void* v_pool, int num_pages,
                                                 const int* page_table, int max_pages, const int* cu_seqlens,
                                                 const int* seq_slots, const int* kv_lens, int num_seqs, int num_tiles,
@@ -669,52 +733,10 @@ extern "C" int rl_attention_prefill_tc_headgate(const void* q, int ldq, const vo
                                                 float scale, int window, int* err, const int* tile_order, int sink,
                                                 const void* gate, int ldg, float softcap, int keep_first, int chunk, int gate_per_head,
                                                 cudaStream_t stream) {
-  RL_REQUIRE(chunk >= 0 && !(chunk > 0 && window > 0), "rl_attention_prefill_tc: a chunked mask and a window exclude one another");
-  RL_REQUIRE(softcap >= 0.f && keep_first >= 0 && scale > 0.f, "rl_attention_prefill_tc: negative soft cap or number of kept first tokens, or a scale that is not positive");
-  const float cap_in = softcap > 0.f ? scale / softcap : 0.f, cap_out = softcap > 0.f ? softcap / scale : 0.f;
-  if (window <= 0) keep_first = 0;
-  RL_REQUIRE(gate == nullptr || (gate_per_head && ldg >= num_heads) || (!gate_per_head && ldg >= num_heads * head_dim && ldg % 8 == 0 && ((uintptr_t)gate & 15) == 0),
-             "rl_attention_prefill_tc: the gate must be 16-byte aligned with a row stride that is a multiple of 8 and holds all heads");
-  RL_REQUIRE(rl_attention_prefill_tc_supported(num_heads, num_kv_heads, head_dim),
-             "rl_attention_prefill_tc: unsupported shape (heads %d, KV heads %d, head_dim %d): needs head_dim 64 or 128",
-             num_heads, num_kv_heads, head_dim);
-  RL_REQUIRE(num_seqs >= 0 && num_tiles >= 0 && num_tokens >= 0 && num_pages > 0 && num_tiles <= 65535, "rl_attention_prefill_tc: bad sizes");
-  RL_REQUIRE(ldq >= num_heads * head_dim && ldq % 8 == 0 && ldo >= num_heads * head_dim && ldo % 8 == 0,
-             "rl_attention_prefill_tc: row strides must be multiples of 8 elements and hold all heads");
-  RL_REQUIRE(((uintptr_t)q & 15) == 0 && ((uintptr_t)out & 15) == 0 && ((uintptr_t)k_pool & 15) == 0 && ((uintptr_t)v_pool & 15) == 0,
-             "rl_attention_prefill_tc: pointers must be 16-byte aligned");
-  RL_REQUIRE(window >= 0 && err != nullptr, "rl_attention_prefill_tc: negative window or null error word");
-  if (num_seqs == 0 || num_tiles == 0) return RL_OK;
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, FaSizes<128>::SMEM);
-    RL_REQUIRE(e == cudaSuccess, "rl_attention_prefill_tc: cannot reserve %d bytes of shared memory: %s", FaSizes<128>::SMEM, cudaGetErrorString(e));
-    e = cudaFuncSetAttribute(attention_prefill_tc_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, FaSizes<64>::SMEM);
-    RL_REQUIRE(e == cudaSuccess, "rl_attention_prefill_tc: cannot reserve %d bytes of shared memory: %s", FaSizes<64>::SMEM, cudaGetErrorString(e));
-    configured = true;
-  }
-  CUtensorMap mq, mk, mv;
-  int rc = fa_make_map(&mq, q, num_tokens, num_heads * head_dim, ldq, TQ);
-  if (rc != RL_OK) return rc;
-  const long long pool_rows = (long long)num_pages * num_kv_heads * RL_PAGE;
-  rc = fa_make_map(&mk, k_pool, pool_rows, head_dim, head_dim, RL_PAGE);
-  if (rc != RL_OK) return rc;
-  rc = fa_make_map(&mv, v_pool, pool_rows, head_dim, head_dim, RL_PAGE);
-  if (rc != RL_OK) return rc;
-  cudaError_t e = head_dim == 128
-      ? rl_launch_pdl(attention_prefill_tc_kernel<128>, dim3(num_heads, num_tiles), dim3(FA_THREADS), (size_t)FaSizes<128>::SMEM, stream,
-                      mq, mk, mv, page_table, max_pages, cu_seqlens, seq_slots, kv_lens, num_seqs,
-                      (__nv_bfloat16*)out, ldo, num_heads, num_kv_heads, scale * 1.4426950408889634f, window, err, tile_order,
-                      sink, (const __nv_bfloat16*)gate, ldg, cap_in, cap_out, keep_first, chunk, gate_per_head)
-      : rl_launch_pdl(attention_prefill_tc_kernel<64>, dim3(num_heads, num_tiles), dim3(FA_THREADS), (size_t)FaSizes<64>::SMEM, stream,
-                      mq, mk, mv, page_table, max_pages, cu_seqlens, seq_slots, kv_lens, num_seqs,
-                      (__nv_bfloat16*)out, ldo, num_heads, num_kv_heads, scale * 1.4426950408889634f, window, err, tile_order,
-                      sink, (const __nv_bfloat16*)gate, ldg, cap_in, cap_out, keep_first, chunk, gate_per_head);
-  if (e != cudaSuccess) {
-    rl_set_error("rl_attention_prefill_tc: launch failed: %s", cudaGetErrorString(e));
-    return RL_ERR_CUDA;
-  }
-  return RL_OK;
+  return rl_attention_prefill_tc_wide(q, ldq, k_pool, v_pool, num_pages, page_table, max_pages, cu_seqlens, seq_slots, kv_lens,
+                                      num_seqs, num_tiles, num_tokens, out, ldo, num_heads, num_kv_heads, head_dim, scale, window,
+                                      err, tile_order, sink, gate, ldg, softcap, keep_first, chunk, gate_per_head, head_dim, nullptr,
+                                      stream);
 }
 
 extern "C" int rl_attention_prefill_tc_shaped(const void* q, int ldq, const void* k_pool, const void* v_pool, int num_pages,

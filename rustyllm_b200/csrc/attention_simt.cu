@@ -33,7 +33,7 @@ attention_simt_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k_
                       const int* __restrict__ slot_of_token, const int* __restrict__ positions,
                       T* __restrict__ out, int ldo, int H, int G, int hd, int vd, float scale, int window,
                       int sink, const T* __restrict__ gate, int ldg, float softcap, int keep_first, int chunk, int ldv,
-                      int gate_per_head) {
+                      int gate_per_head, const float* __restrict__ sinks) {
   __shared__ float s_acc[ATT_WARPS][NE * 32];
   __shared__ float s_max[ATT_WARPS], s_sum[ATT_WARPS];
   const int m = blockIdx.x, h = blockIdx.y;
@@ -108,11 +108,14 @@ attention_simt_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k_
     if (d < vd) s_acc[warp][d] = acc[e];
   }
   __syncthreads();
-  // sink: one more term in the denominator with score 0 and no value, p_j = e^{s_j} / (1 + sum e^{s_t})
-  float M = sink ? 0.f : -INFINITY;
+  // sink: one more term in the denominator without a value, p_j = e^{s_j} / (e^{z} + sum e^{s_t}), of score z = 0 or the
+  // head's own (sinks[h])
+  const bool has_sink = sink || sinks != nullptr;
+  const float sink_score = sinks ? sinks[h] : 0.f;
+  float M = has_sink ? sink_score : -INFINITY;
 #pragma unroll
   for (int w = 0; w < ATT_WARPS; ++w) M = fmaxf(M, s_max[w]);
-  float wgt[ATT_WARPS], L = sink ? expf(-M) : 0.f;
+  float wgt[ATT_WARPS], L = has_sink ? expf(sink_score - M) : 0.f;
 #pragma unroll
   for (int w = 0; w < ATT_WARPS; ++w) {
     wgt[w] = s_max[w] > -INFINITY ? expf(s_max[w] - M) : 0.f;
@@ -146,12 +149,14 @@ attention_simt_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k_
 // chunk > 0 (instead of a window): a query at position p sees positions [p - p % chunk, p].  value_stride: elements
 // from one value row to the next (0: value_dim); with value_stride = head_dim and v_pool = k_pool the values are the
 // first value_dim elements of the key rows.  gate_per_head != 0: gate is [M, ldg] with one number a head.
+// sinks (float [num_heads], may be null): the sink term has this score for each head (no scale, no soft cap).
 extern "C" int rl_attention_simt_shaped(const void* q, int ldq, const void* k_pool, const void* v_pool,
                                         int dtype, const int* page_table, int max_pages,
                                         const int* slot_of_token, const int* positions, void* out, int ldo,
                                         int num_tokens, int num_heads, int num_kv_heads, int head_dim, int value_dim,
                                         float scale, int window, int sink, const void* gate, int ldg, float softcap,
-                                        int keep_first, int chunk, int value_stride, int gate_per_head, cudaStream_t stream) {
+                                        int keep_first, int chunk, int value_stride, int gate_per_head, const float* sinks,
+                                        cudaStream_t stream) {
   RL_REQUIRE(chunk >= 0 && !(chunk > 0 && window > 0), "rl_attention_simt: a chunked mask and a window exclude one another");
   RL_REQUIRE(value_stride == 0 || value_stride >= value_dim, "rl_attention_simt: value rows %d apart are shorter than a value (%d)",
              value_stride, value_dim);
@@ -173,7 +178,7 @@ extern "C" int rl_attention_simt_shaped(const void* q, int ldq, const void* k_po
   attention_simt_kernel<T, NE><<<grid, ATT_WARPS * 32, 0, stream>>>(                                                      \
       (const T*)q, ldq, (const T*)k_pool, (const T*)v_pool, page_table, max_pages, slot_of_token, positions, (T*)out, ldo, \
       num_heads, num_kv_heads, head_dim, value_dim, scale, window, sink, (const T*)gate, ldg, softcap, keep_first, chunk,  \
-      ldv, gate_per_head)
+      ldv, gate_per_head, sinks)
   if (dtype == RL_F32) {
     if (wide) RL_ATT_SIMT_LAUNCH(float, 32); else RL_ATT_SIMT_LAUNCH(float, 8);
   } else if (dtype == RL_BF16) {
@@ -194,7 +199,7 @@ extern "C" int rl_attention_simt_masked(const void* q, int ldq, const void* k_po
                                         int keep_first, cudaStream_t stream) {
   return rl_attention_simt_shaped(q, ldq, k_pool, v_pool, dtype, page_table, max_pages, slot_of_token, positions, out, ldo,
                                   num_tokens, num_heads, num_kv_heads, head_dim, value_dim, scale, window, sink, gate, ldg, softcap,
-                                  keep_first, 0, 0, 0, stream);
+                                  keep_first, 0, 0, 0, nullptr, stream);
 }
 
 extern "C" int rl_attention_simt_gated(const void* q, int ldq, const void* k_pool, const void* v_pool,

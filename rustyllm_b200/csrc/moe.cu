@@ -5,6 +5,7 @@
 //            weights = softmax over the chosen logits only
 //   expert : y_e = Wdown_e (silu(Wgate_e h) * (Wup_e h))
 //   output : residual += sum_c weight_c * y_{e_c}     (choices in the order of falling logits)
+//   or, weights on the input: y_e = expert(weight * h), residual += sum_c y_{e_c}
 //
 // The gate's activation is an argument: 0 silu(g) * u; 1 g = min(g, limit), u = clamp(u, -limit, limit),
 // g sigmoid(alpha g) (u + 1).
@@ -376,7 +377,8 @@ extern "C" int rl_moe_route_sigmoid(const void* x, int ldx, const void* router, 
 template <typename T>
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_gate_up_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ wgu, const int* __restrict__ ids,
-                   int d, int F, int top, T* __restrict__ h, int interleaved, int act, float limit, float alpha) {
+                   int d, int F, int top, T* __restrict__ h, int interleaved, int act, float limit, float alpha,
+                   const float* __restrict__ in_weights) {
   extern __shared__ float s_x[];          // [d]
   rl_pdl_trigger();
   rl_pdl_wait();
@@ -406,6 +408,10 @@ moe_gate_up_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ wgu, 
   g = rl_warp_sum(g);
   u = rl_warp_sum(u);
   if (lane == 0) {
+    if (in_weights) {          // the expert reads weight * h: both products scale with it
+      g *= in_weights[pair];
+      u *= in_weights[pair];
+    }
     if (act == 1) {
       g = fminf(g, limit);
       u = fminf(fmaxf(u, -limit), limit);
@@ -445,16 +451,20 @@ moe_down_kernel(const T* __restrict__ h, const T* __restrict__ wd, const int* __
       for (int i = lane; i < F; i += 32) part = fmaf(rl_ld(hr + i), rl_ld(w + i), part);
     }
     part = rl_warp_sum(part);
-    y = fmaf(weights[(size_t)m * top + c], part, y);
+    y = fmaf(weights ? weights[(size_t)m * top + c] : 1.f, part, y);
   }
   if (lane == 0) residual[(size_t)m * d + r] += y;
 }
 
 // x [M, ldx]; gate_up [E, 2, F, d], or with `interleaved` [E, F, 2, d] (gate_r, up_r in turn); down [E, d, F]; ids, weights [M, top] (from rl_moe_route);
-// h [M * top, F] scratch in the same dtype; residual [M, d] float, added into.
+// h [M * top, F] scratch in the same dtype; residual [M, d] float, added into.  weigh_input != 0: the weight multiplies the
+// expert's input, not its output.
 extern "C" int rl_moe_experts(const void* x, int ldx, const void* gate_up, const void* down, int dtype, const int* ids,
                               const float* weights, int num_tokens, int hidden, int expert_ff, int num_experts, int top,
-                              int interleaved, int act, float limit, float alpha, void* h, float* residual, cudaStream_t stream) {
+                              int interleaved, int act, float limit, float alpha, int weigh_input, void* h, float* residual,
+                              cudaStream_t stream) {
+  const float* wi = weigh_input ? weights : nullptr;      // on the way in
+  const float* wo = weigh_input ? nullptr : weights;      // on the way out
   RL_REQUIRE(act == 0 || act == 1, "rl_moe_experts: unknown activation %d", act);
   RL_REQUIRE(num_tokens >= 0 && hidden > 0 && expert_ff > 0 && num_experts > 0 && top > 0,
              "rl_moe_experts: bad sizes M=%d d=%d F=%d E=%d top=%d", num_tokens, hidden, expert_ff, num_experts, top);
@@ -470,14 +480,16 @@ extern "C" int rl_moe_experts(const void* x, int ldx, const void* gate_up, const
     const size_t smem = (size_t)hidden * sizeof(float);
     if (dtype == RL_F32) {
       rl_launch_pdl(moe_gate_up_kernel<float>, g1, MOE_THREADS, smem, stream, (const float*)x + (size_t)m0 * ldx, ldx, (const float*)gate_up,
-                    ids + p0, hidden, expert_ff, top, (float*)h + (size_t)p0 * expert_ff, interleaved, act, limit, alpha);
+                    ids + p0, hidden, expert_ff, top, (float*)h + (size_t)p0 * expert_ff, interleaved, act, limit, alpha,
+                    wi ? wi + p0 : nullptr);
       rl_launch_pdl(moe_down_kernel<float>, g2, MOE_THREADS, 0, stream, (const float*)h + (size_t)p0 * expert_ff, (const float*)down,
-                    ids + p0, weights + p0, hidden, expert_ff, top, residual + (size_t)m0 * hidden);
+                    ids + p0, wo ? wo + p0 : nullptr, hidden, expert_ff, top, residual + (size_t)m0 * hidden);
     } else if (dtype == RL_BF16) {
       rl_launch_pdl(moe_gate_up_kernel<__nv_bfloat16>, g1, MOE_THREADS, smem, stream, (const __nv_bfloat16*)x + (size_t)m0 * ldx, ldx,
-                    (const __nv_bfloat16*)gate_up, ids + p0, hidden, expert_ff, top, (__nv_bfloat16*)h + (size_t)p0 * expert_ff, interleaved, act, limit, alpha);
+                    (const __nv_bfloat16*)gate_up, ids + p0, hidden, expert_ff, top, (__nv_bfloat16*)h + (size_t)p0 * expert_ff, interleaved, act, limit, alpha,
+                    wi ? wi + p0 : nullptr);
       rl_launch_pdl(moe_down_kernel<__nv_bfloat16>, g2, MOE_THREADS, 0, stream, (const __nv_bfloat16*)h + (size_t)p0 * expert_ff,
-                    (const __nv_bfloat16*)down, ids + p0, weights + p0, hidden, expert_ff, top, residual + (size_t)m0 * hidden);
+                    (const __nv_bfloat16*)down, ids + p0, wo ? wo + p0 : nullptr, hidden, expert_ff, top, residual + (size_t)m0 * hidden);
     } else {
       RL_REQUIRE(false, "rl_moe_experts: unknown dtype %d", dtype);
     }
@@ -491,7 +503,7 @@ extern "C" int rl_moe_experts(const void* x, int ldx, const void* gate_up, const
 // pairs are put in the order of their experts, every expert's rows padded to whole token tiles of `bt` rows, so
 // that a tile meets one expert's matrix.
 //   plan   : row[p] = the pair's row; tile_group[t] = the expert of tile t, or -1 for a tile that holds no pair
-//   gather : xs[row[p], :] = x[p / top, :]
+//   gather : xs[row[p], :] = x[p / top, :]            (times weights[p], where the weights are the input's)
 //   (grouped products: gate and up with the activation in the epilogue, then down, into y [rows, d] float)
 //   combine: residual[m, :] += sum_c weights[m, c] * y[row[m * top + c], :]   (choices in their order)
 // Which row a pair gets within its expert depends on timing; no result does: a row of a product depends on that
@@ -528,13 +540,28 @@ moe_plan_kernel(const int* __restrict__ ids, int pairs, int E, int bt, int max_t
 }
 
 __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const int* __restrict__ row, int top, int d,
-                                  __nv_bfloat16* __restrict__ xs) {
+                                  const float* __restrict__ in_weights, __nv_bfloat16* __restrict__ xs) {
   rl_pdl_trigger();
   rl_pdl_wait();
   const int p = blockIdx.x;
   const __nv_bfloat16* src = x + (size_t)(p / top) * ldx;
   __nv_bfloat16* dst = xs + (size_t)row[p] * d;
-  for (int i = threadIdx.x; i < d / 8; i += blockDim.x)          // d is a multiple of 8, rows 16-byte aligned
+  // d is a multiple of 8, rows 16-byte aligned
+  if (in_weights) {
+    const float w = in_weights[p];
+    for (int i = threadIdx.x; i < d / 8; i += blockDim.x) {
+      uint4 v = reinterpret_cast<const uint4*>(src)[i];
+      __nv_bfloat162* e = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 f = __bfloat1622float2(e[k]);
+        e[k] = __floats2bfloat162_rn(w * f.x, w * f.y);
+      }
+      reinterpret_cast<uint4*>(dst)[i] = v;
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < d / 8; i += blockDim.x)
     reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
 }
 
@@ -547,7 +574,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
   for (int i = 4 * threadIdx.x; i < d; i += 4 * blockDim.x) {
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int c = 0; c < top; ++c) {
-      const float w = weights[(size_t)m * top + c];
+      const float w = weights ? weights[(size_t)m * top + c] : 1.f;
       const float4 v = __ldcs(reinterpret_cast<const float4*>(y + (size_t)row[(size_t)m * top + c] * d + i));
       acc.x = fmaf(w, v.x, acc.x); acc.y = fmaf(w, v.y, acc.y); acc.z = fmaf(w, v.z, acc.z); acc.w = fmaf(w, v.w, acc.w);
     }
@@ -573,10 +600,11 @@ extern "C" int rl_moe_plan(const int* ids, int pairs, int num_experts, int bt, i
   return RL_OK;
 }
 
-extern "C" int rl_moe_gather(const void* x, int ldx, const int* row, int pairs, int top, int hidden, void* xs, cudaStream_t stream) {
+extern "C" int rl_moe_gather(const void* x, int ldx, const int* row, int pairs, int top, int hidden, const float* in_weights, void* xs,
+                             cudaStream_t stream) {
   RL_REQUIRE(pairs > 0 && top > 0 && hidden % 8 == 0 && ldx % 8 == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)xs & 15) == 0,
              "rl_moe_gather: rows must be 16-byte aligned and a multiple of 8 long");
-  rl_launch_pdl(moe_gather_kernel, pairs, 128, 0, stream, (const __nv_bfloat16*)x, ldx, row, top, hidden, (__nv_bfloat16*)xs);
+  rl_launch_pdl(moe_gather_kernel, pairs, 128, 0, stream, (const __nv_bfloat16*)x, ldx, row, top, hidden, in_weights, (__nv_bfloat16*)xs);
   RL_LAUNCH_CHECK("rl_moe_gather");
   return RL_OK;
 }

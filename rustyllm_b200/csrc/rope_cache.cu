@@ -203,6 +203,68 @@ rope_kv_write_bf16_pairs_kernel(__nv_bfloat16* __restrict__ qkv, int ld, const i
   }
 }
 
+// The same pairing where the general shape asks for more: a part of the head rotated (rotary width a multiple of 16), value
+// heads of another width, queries alone (G = 0, nothing cached).  A thread rotates eight pairs, or copies eight elements of
+// a key's unrotated tail or of a value; the token's sines and cosines once a CTA.
+__global__ void __launch_bounds__(ROPE_THREADS)
+rope_kv_write_bf16_halves_kernel(__nv_bfloat16* __restrict__ qkv, int ld, const int* __restrict__ positions,
+                                 const int* __restrict__ slot_of_token, const int* __restrict__ page_table, int max_pages,
+                                 const float* __restrict__ inv_freq, int H, int G, int hd, int vd, int rot,
+                                 __nv_bfloat16* __restrict__ k_pool, __nv_bfloat16* __restrict__ v_pool) {
+  __shared__ float2 cs[128];                              // (cos, sin) of the token's rot / 2 <= 128 angles
+  rl_pdl_trigger();
+  rl_pdl_wait();
+  const int m = blockIdx.x;
+  const int pos = positions[m];
+  __nv_bfloat16* row = qkv + (size_t)m * ld;
+  size_t dst_k = 0, dst_v = 0;
+  if (G > 0) {
+    const int page = page_table[(size_t)slot_of_token[m] * max_pages + pos / RL_PAGE];
+    dst_k = ((size_t)page * G) * RL_PAGE * hd + (size_t)(pos % RL_PAGE) * hd;
+    dst_v = ((size_t)page * G) * RL_PAGE * vd + (size_t)(pos % RL_PAGE) * vd;
+  }
+  const int half = rot / 2;
+  for (int i = threadIdx.x; i < half; i += ROPE_THREADS) {
+    float sn, c;
+    sincosf((float)pos * inv_freq[i], &sn, &c);
+    cs[i] = make_float2(c, sn);
+  }
+  __syncthreads();
+  const int pairs8 = half / 8, tail8 = (hd - rot) / 8, v8 = vd / 8;
+  const int n_rot = (H + G) * pairs8, n_tail = G * tail8, n_v = G * v8;
+  for (int idx = threadIdx.x; idx < n_rot + n_tail + n_v; idx += ROPE_THREADS) {
+    if (idx < n_rot) {
+      const int hs = idx / pairs8, i = (idx % pairs8) * 8;
+      __nv_bfloat16* x = row + (size_t)hs * hd;
+      const uint4 lo = *reinterpret_cast<const uint4*>(x + i);
+      const uint4 hi = *reinterpret_cast<const uint4*>(x + i + half);
+      const __nv_bfloat162* l2 = reinterpret_cast<const __nv_bfloat162*>(&lo);
+      const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&hi);
+      uint4 olo, ohi;
+      __nv_bfloat162* ol = reinterpret_cast<__nv_bfloat162*>(&olo);
+      __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&ohi);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 a = __bfloat1622float2(l2[k]), b = __bfloat1622float2(h2[k]);
+        const float2 t0 = cs[i + 2 * k], t1 = cs[i + 2 * k + 1];
+        ol[k] = __floats2bfloat162_rn(a.x * t0.x - b.x * t0.y, a.y * t1.x - b.y * t1.y);
+        oh[k] = __floats2bfloat162_rn(a.x * t0.y + b.x * t0.x, a.y * t1.y + b.y * t1.x);
+      }
+      __nv_bfloat16* d = hs < H ? x : k_pool + dst_k + (size_t)(hs - H) * RL_PAGE * hd;
+      *reinterpret_cast<uint4*>(d + i) = olo;
+      *reinterpret_cast<uint4*>(d + i + half) = ohi;
+    } else if (idx < n_rot + n_tail) {
+      const int g = (idx - n_rot) / tail8, i = rot + ((idx - n_rot) % tail8) * 8;
+      *reinterpret_cast<uint4*>(k_pool + dst_k + (size_t)g * RL_PAGE * hd + i) =
+          *reinterpret_cast<const uint4*>(row + (size_t)(H + g) * hd + i);
+    } else {
+      const int at = idx - n_rot - n_tail, g = at / v8, i = (at % v8) * 8;
+      *reinterpret_cast<uint4*>(v_pool + dst_v + (size_t)g * RL_PAGE * vd + i) =
+          *reinterpret_cast<const uint4*>(row + (size_t)(H + G) * hd + (size_t)g * vd + i);
+    }
+  }
+}
+
 // No rotation at all (rotary width 0): keys and values go to their pages as they are, 16 bytes a thread;
 // the queries stay where they are.  One CTA a token; any dtype (bytes are copied).
 __global__ void __launch_bounds__(ROPE_THREADS)
@@ -226,7 +288,7 @@ kv_write_copy_kernel(const uint4* __restrict__ qkv, int ld16, const int* __restr
 // heads of value_dim (even; it may differ from head_dim).  Queries are rotated in place;
 // rotated keys go to k_pool [pages, G, RL_PAGE, head_dim] and the values to v_pool
 // [pages, G, RL_PAGE, value_dim] (same dtype as qkv).  With k_pool == nullptr nothing is
-// cached and the keys are rotated in place as well.
+// cached and the keys are rotated in place as well.  num_kv_heads may be 0 then: queries alone.
 //
 // rl_rope_kv_write_mixed: the same, and where `v_other` is given ([M, ld_other] in the same dtype, G value heads a
 // row, e.g. the values an earlier layer made of the same tokens) the values become (1 - lam) v + lam v_other with
@@ -236,7 +298,7 @@ extern "C" int rl_rope_kv_write_mixed(void* qkv, int dtype, int ld, const int* p
                                       const float* inv_freq, int num_tokens, int num_heads, int num_kv_heads,
                                       int head_dim, int value_dim, int rotary_dim, int interleaved, void* k_pool,
                                       void* v_pool, const void* v_other, int ld_other, const float* v_mix, cudaStream_t stream) {
-  RL_REQUIRE(num_tokens >= 0 && num_heads > 0 && num_kv_heads > 0, "rl_rope_kv_write: bad sizes");
+  RL_REQUIRE(num_tokens >= 0 && num_heads > 0 && (num_kv_heads > 0 || (num_kv_heads == 0 && k_pool == nullptr)), "rl_rope_kv_write: bad sizes");
   RL_REQUIRE(head_dim > 0 && head_dim <= 256, "rl_rope_kv_write: head_dim %d outside (0, 256]", head_dim);
   RL_REQUIRE(rotary_dim >= 0 && rotary_dim <= head_dim && rotary_dim % 2 == 0,
              "rl_rope_kv_write: rotary_dim %d must be even and <= head_dim %d", rotary_dim, head_dim);
@@ -269,6 +331,12 @@ extern "C" int rl_rope_kv_write_mixed(void* qkv, int dtype, int ld, const int* p
     rl_launch_pdl(rope_kv_write_bf16_pairs_kernel, dim3(num_tokens), threads, 0, stream, (__nv_bfloat16*)qkv, ld, positions, slot_of_token,
                   page_table, max_pages, inv_freq, num_heads, num_kv_heads, head_dim, value_dim, rotary_dim, (__nv_bfloat16*)k_pool,
                   (__nv_bfloat16*)v_pool, (const __nv_bfloat16*)v_other, ld_other, v_mix);
+  else if (v_other == nullptr && dtype == RL_BF16 && (write_cache || num_kv_heads == 0) && !interleaved && rotary_dim > 0 && rotary_dim % 16 == 0 &&
+           head_dim % 8 == 0 && value_dim % 8 == 0 && ld % 8 == 0 && ((uintptr_t)qkv & 15) == 0 && ((uintptr_t)k_pool & 15) == 0 &&
+           ((uintptr_t)v_pool & 15) == 0)
+    rl_launch_pdl(rope_kv_write_bf16_halves_kernel, dim3(num_tokens), threads, 0, stream, (__nv_bfloat16*)qkv, ld, positions, slot_of_token,
+                  page_table, max_pages, inv_freq, num_heads, num_kv_heads, head_dim, value_dim, rotary_dim, (__nv_bfloat16*)k_pool,
+                  (__nv_bfloat16*)v_pool);
   else if (dtype == RL_F32)
     rl_launch_pdl(rope_kv_write_kernel<float>, grid, threads, 0, stream,
         (float*)qkv, ld, positions, slot_of_token, page_table, max_pages, inv_freq, num_heads,

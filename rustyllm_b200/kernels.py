@@ -42,7 +42,14 @@ _SIGNATURES = {
     "rl_random_fill": [_c_void_p, _c_int, _c_ll, ctypes.c_ulonglong, _c_float, _c_float, _c_void_p],
     "rl_gemm_simt": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
                      _c_int, _c_int, _c_void_p],
-    "rl_layer_norm": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_float, _c_void_p],
+    "rl_layer_norm": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_float, _c_void_p],
+    "rl_branch_join": [_c_void_p, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
+                       _c_void_p, _c_void_p, _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
+    "rl_gated_linear_scan": [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_float, _c_float,
+                             _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    "rl_gated_delta_scan": [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int,
+                            _c_void_p, _c_void_p, _c_float, _c_float, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll, _c_void_p, _c_int,
+                            _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "rl_token_shift_mix": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll,
                            _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
     "rl_tanh_cast": [_c_void_p, _c_void_p, _c_int, _c_ll, _c_void_p],
@@ -72,7 +79,7 @@ _SIGNATURES = {
                                  _c_int, _c_void_p, _c_int, _c_float, _c_int, _c_void_p],
     "rl_attention_simt_shaped": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p,
                                  _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int,
-                                 _c_int, _c_void_p, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+                                 _c_int, _c_void_p, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "rl_attention_shared_key_supported": [_c_int, _c_int, _c_int],
     "rl_attention_shared_key": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
                                 _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void_p,
@@ -127,9 +134,9 @@ _SIGNATURES = {
                      _c_void_p],
     "rl_moe_select": [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p],
     "rl_moe_experts": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
-                       _c_int, _c_int, _c_int, _c_float, _c_float, _c_void_p, _c_void_p, _c_void_p],
+                       _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p],
     "rl_moe_plan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p],
-    "rl_moe_gather": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+    "rl_moe_gather": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p],
     "rl_moe_combine": [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "rl_gemm_tc_grouped": [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
                            _c_void_p, _c_int, _c_int, _c_float, _c_float, _c_void_p],
@@ -161,6 +168,13 @@ _SIGNATURES = {
     "rl_attention_decode_headgate": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
                                      _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int,
                                      _c_int, _c_void_p, _c_int, _c_float, _c_int, _c_int, _c_void_p],
+    "rl_attention_decode_wide": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
+                                 _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int,
+                                 _c_int, _c_void_p, _c_int, _c_float, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+    "rl_attention_prefill_tc_wide": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p,
+                                     _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float,
+                                     _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_int, _c_int, _c_int,
+                                     _c_int, _c_void_p, _c_void_p],
     "rl_attention_prefill_tc_headgate": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p,
                                          _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float,
                                          _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_int, _c_int, _c_int, _c_void_p],
@@ -169,6 +183,10 @@ _SIGNATURES = {
     "rl_attention_decode_places": [_c_int],
     "rl_attention_decode_ring_bytes": [_c_int],
     "rl_attention_decode_supported": [_c_int, _c_int, _c_int],
+    "rl_attention_decode_places_shaped": [_c_int, _c_int],
+    "rl_attention_decode_ring_bytes_shaped": [_c_int, _c_int],
+    "rl_attention_decode_supported_shaped": [_c_int, _c_int, _c_int, _c_int],
+    "rl_attention_prefill_tc_supported_shaped": [_c_int, _c_int, _c_int, _c_int],
     "rl_attention_prefill": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
                              _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p],
     "rl_attention_prefill_supported": [_c_int, _c_int, _c_int],
@@ -387,12 +405,13 @@ def moe_select(logits: torch.Tensor, top: int, ids: torch.Tensor, weights: torch
 
 
 def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-                residual: torch.Tensor, interleaved: bool = False, act=None) -> None:
+                residual: torch.Tensor, interleaved: bool = False, act=None, weigh_input: bool = False) -> None:
     """residual[m] += sum_c weights[m, c] * down[e] (silu(gate[e] x[m]) * (up[e] x[m])), e = ids[m, c], on the
     CUDA cores (any sizes, float32 or bfloat16 storage): every (token, choice) pair reads its expert's rows,
     which is what a step of few tokens needs.  gate_up: [E, 2, F, d] (an expert's gate rows, then its up
     rows) or, ``interleaved``, [E, F, 2, d] (gate_r, up_r in turn); down: [E, d, F].  ``act`` (limit, alpha): the clamped
-    gate instead of silu, g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    gate instead of silu, g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).
+    ``weigh_input``: the weight multiplies the expert's input instead of its output."""
     limit, alpha = act if act is not None else (0.0, 0.0)
     _need(x, "x", contiguous=False); _need(gate_up, "gate_up", x.dtype); _need(down, "down", x.dtype)
     _need(ids, "ids", torch.int32); _need(weights, "weights", torch.float32); _need(residual, "residual", torch.float32)
@@ -407,7 +426,8 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
     h = torch.empty((M * top, F), dtype=x.dtype, device=x.device)
     _check(library().rl_moe_experts(x.data_ptr(), x.stride(0) if M > 1 else d, gate_up.data_ptr(), down.data_ptr(), _dt(x),
                                     ids.data_ptr(), weights.data_ptr(), M, d, F, E, top, int(bool(interleaved)), int(act is not None),
-                                    float(limit), float(alpha), h.data_ptr(), residual.data_ptr(), _stream()), "rl_moe_experts")
+                                    float(limit), float(alpha), int(bool(weigh_input)), h.data_ptr(), residual.data_ptr(), _stream()),
+           "rl_moe_experts")
     _count(2)
 
 
@@ -426,13 +446,14 @@ def moe_experts_grouped_supported(x: torch.Tensor, gate_up: torch.Tensor, down: 
 
 
 def moe_experts_grouped(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-                        residual: Optional[torch.Tensor], act=None):
+                        residual: Optional[torch.Tensor], act=None, weigh_input: bool = False):
     """The same sum as ``moe_experts`` on the tensor cores, for steps of many tokens: the (token, choice) pairs
     are ordered by expert (every expert's rows padded to whole token tiles), gate and up run as one grouped
     product with the activation in its epilogue, down as a second one, and the choices of a token are added
     into the residual in their order.  gate_up: [E, F, 2, d] (gate_r, up_r in turn), down: [E, d, F], bf16.  ``act``: see
     ``moe_experts``.  Without ``residual`` nothing is added: returns (y float32 [rows, d], row int32 [M * top]), the
-    experts' unweighted outputs and where each (token, choice) pair's row lies."""
+    experts' unweighted outputs and where each (token, choice) pair's row lies.  ``weigh_input``: the weight multiplies the
+    expert's input (rounded to bfloat16), and the outputs are summed as they are."""
     _need(x, "x", torch.bfloat16, contiguous=False); _need(gate_up, "gate_up", torch.bfloat16); _need(down, "down", torch.bfloat16)
     _need(ids, "ids", torch.int32); _need(weights, "weights", torch.float32)
     limit, alpha = act if act is not None else (0.0, 0.0)
@@ -452,7 +473,8 @@ def moe_experts_grouped(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tens
     y = torch.empty((rows, d), dtype=torch.float32, device=dev)
     lib, st, err = library(), _stream(), _tc_error_word(dev).data_ptr()
     _check(lib.rl_moe_plan(ids.data_ptr(), pairs, E, bt, tiles, row.data_ptr(), tile_group.data_ptr(), st), "rl_moe_plan")
-    _check(lib.rl_moe_gather(x.data_ptr(), x.stride(0) if M > 1 else d, row.data_ptr(), pairs, top, d, xs.data_ptr(), st), "rl_moe_gather")
+    _check(lib.rl_moe_gather(x.data_ptr(), x.stride(0) if M > 1 else d, row.data_ptr(), pairs, top, d,
+                             weights.data_ptr() if weigh_input else None, xs.data_ptr(), st), "rl_moe_gather")
     _check(lib.rl_gemm_tc_grouped(xs.data_ptr(), gate_up.data_ptr(), h.data_ptr(), OUT_SWIGLU if act is None else OUT_CLAMPED, rows,
                                   2 * F, d, d, F, err, tile_group.data_ptr(), E, bt, float(limit), float(alpha), st), "rl_gemm_tc_grouped")
     _check(lib.rl_gemm_tc_grouped(h.data_ptr(), down.data_ptr(), y.data_ptr(), OUT_F32, rows, d, F, F, d, err,
@@ -462,7 +484,7 @@ def moe_experts_grouped(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tens
         return y, row
     _need(residual, "residual", torch.float32)
     assert residual.shape == (M, d)
-    _check(lib.rl_moe_combine(y.data_ptr(), row.data_ptr(), weights.data_ptr(), M, top, d, residual.data_ptr(), st), "rl_moe_combine")
+    _check(lib.rl_moe_combine(y.data_ptr(), row.data_ptr(), None if weigh_input else weights.data_ptr(), M, top, d, residual.data_ptr(), st), "rl_moe_combine")
     _count(5)
 
 
@@ -575,12 +597,14 @@ def rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, slot_of_token: tor
                   v_other: Optional[torch.Tensor] = None, v_mix: Optional[torch.Tensor] = None) -> None:
     """Rotates the query and key heads of qkv ([M, H*hd + G*hd + G*vd]) in place and writes keys
     and values at their tokens' places of the paged pools.  ``value_dim`` (default: head_dim)
-    is the width of a value head.  ``v_other`` [M, G*vd] (a view is fine) with ``v_mix`` (a float32 scalar on the
+    is the width of a value head; without keys and values (``num_kv_heads`` 0, no pools) the queries alone are rotated.
+    ``v_other`` [M, G*vd] (a view is fine) with ``v_mix`` (a float32 scalar on the
     device): the values become (1 - v_mix) v + v_mix v_other, in 32-bit, before they are cached."""
     vd = head_dim if value_dim is None else value_dim
     _need(qkv, "qkv", contiguous=False); _need(positions, "positions", torch.int32)
     _need(inv_freq, "inv_freq", torch.float32)
     M = qkv.shape[0]
+    assert num_kv_heads > 0 or k_pool is None
     assert qkv.stride(1) == 1 and (M == 1 or qkv.stride(0) >= qkv.shape[1])
     if k_pool is not None:
         _need(k_pool, "k_pool", qkv.dtype); _need(v_pool, "v_pool", qkv.dtype)
@@ -608,7 +632,7 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
                    num_heads: int, num_kv_heads: int, head_dim: int, scale: float, window: int = 0,
                    value_dim: Optional[int] = None, sink: bool = False, gate: Optional[torch.Tensor] = None,
                    softcap: float = 0.0, keep_first: int = 0, chunk: int = 0, values_in_keys: bool = False,
-                   gate_per_head: bool = False) -> None:
+                   gate_per_head: bool = False, sinks: Optional[torch.Tensor] = None) -> None:
     """q: [M, >= H*hd] (a view into the qkv buffer is fine), out: [M, H*vd] where vd is
     ``value_dim`` (default: head_dim), the width of a value head.  ``sink``: the softmax's
     denominator has one more term of score 0 (and no value).  ``gate`` [M, H*vd] (a view is
@@ -616,7 +640,8 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
     (scale included) becomes softcap * tanh(s / softcap).  ``keep_first``: with a window, positions
     [0, keep_first) stay visible after the window has passed them.  ``chunk`` > 0 (instead of a window): a query at
     position p sees positions [p - p % chunk, p].  ``values_in_keys``: the values are the first ``value_dim`` elements
-    of the key rows (``v_pool`` is not read).  ``gate_per_head``: ``gate`` is [M, H], one number a head."""
+    of the key rows (``v_pool`` is not read).  ``gate_per_head``: ``gate`` is [M, H], one number a head.  ``sinks`` (float32
+    [H]): the extra term of the denominator has the score sinks[h] instead of 0."""
     vd = head_dim if value_dim is None else value_dim
     if values_in_keys:
         assert vd <= head_dim
@@ -637,15 +662,25 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
         page_table.shape[1], slot_of_token.data_ptr(), positions.data_ptr(), out.data_ptr(), out.stride(0),
         M, num_heads, num_kv_heads, head_dim, vd, float(scale), int(window), int(bool(sink)), _ptr(gate), ldg,
         float(softcap or 0.0), int(keep_first or 0), int(chunk or 0), head_dim if values_in_keys else 0,
-        int(bool(gate_per_head)), _stream()),
+        int(bool(gate_per_head)), _sinks(sinks, num_heads), _stream()),
         "rl_attention_simt")
     _count()
 
 
+def _sinks(sinks: Optional[torch.Tensor], num_heads: int):
+    if sinks is None:
+        return None
+    _need(sinks, "sinks", torch.float32)
+    assert sinks.numel() == num_heads
+    return sinks.data_ptr()
+
+
 def layer_norm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float, rows: Optional[torch.Tensor] = None,
-               weight2: Optional[torch.Tensor] = None, out2: Optional[torch.Tensor] = None) -> None:
+               weight2: Optional[torch.Tensor] = None, out2: Optional[torch.Tensor] = None,
+               bias: Optional[torch.Tensor] = None) -> None:
     """out[r] = (x[r] - mean) / sqrt(mean of squared deviations + eps) * weight (x[rows[r]] if rows is given); with
-    ``weight2`` and ``out2``: also the same row's norm times the second weight, from one read of x."""
+    ``weight2`` and ``out2``: also the same row's norm times the second weight, from one read of x.  ``bias`` [d]: added to
+    ``out`` (not to ``out2``)."""
     _need(x, "x", torch.float32); _need(weight, "weight", torch.float32); _need(out, "out")
     d = x.shape[-1]
     n = out.shape[0]
@@ -660,7 +695,10 @@ def layer_norm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: fl
     if out2 is not None:
         _need(weight2, "weight2", torch.float32); _need(out2, "out2", out.dtype)
         assert weight2.numel() == d and out2.shape == out.shape
-    _check(library().rl_layer_norm(x.data_ptr(), weight.data_ptr(), out.data_ptr(), _ptr(weight2), _ptr(out2), _dt(out), _ptr(rows), n, d,
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        assert bias.numel() == d
+    _check(library().rl_layer_norm(x.data_ptr(), weight.data_ptr(), _ptr(bias), out.data_ptr(), _ptr(weight2), _ptr(out2), _dt(out), _ptr(rows), n, d,
                                    float(eps), _stream()), "rl_layer_norm")
     _count()
 
@@ -1101,6 +1139,105 @@ def channel_decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, wlog: 
     _count()
 
 
+def gated_linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, tau: float, q_scale: float, out: torch.Tensor,
+                      state: torch.Tensor, cu_seqlens: torch.Tensor, seq_slots: torch.Tensor, num_heads: int, dk: int, dv: int) -> None:
+    """S_t = diag(a_t) S_{t-1} + k_t v_t^T with a_t = sigmoid(z_t)^(1/tau), out_t = S_t^T (q_scale q_t), for every head of
+    every sequence of the step; the state (float [H, dv, dk] a slot) is read from and left in ``state``.  q, k [M, H * dk],
+    v [M, H * dv] (views are fine), z float32 [M, H * dk], out float32 [M, H * dv]."""
+    for t, name in ((q, "q"), (k, "k"), (v, "v")):
+        _need(t, name, q.dtype, contiguous=False)
+        assert t.stride(1) == 1
+    _need(out, "out", torch.float32); _need(z, "z", torch.float32, contiguous=False)
+    _need(cu_seqlens, "cu_seqlens", torch.int32); _need(seq_slots, "seq_slots", torch.int32)
+    M = out.shape[0]
+    assert out.shape == (M, num_heads * dv) and q.shape == (M, num_heads * dk) and k.shape == q.shape and v.shape == (M, num_heads * dv)
+    assert z.shape == (M, num_heads * dk) and z.stride(1) == 1
+    sp, ss = _state_args(state)
+    assert state.shape[1] >= 4 * num_heads * dk * dv
+    _check(library().rl_gated_linear_scan(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), _dt(q),
+                                          z.data_ptr(), z.stride(0) if M > 1 else num_heads * dk, float(tau), float(q_scale),
+                                          cu_seqlens.data_ptr(), seq_slots.data_ptr(), seq_slots.numel(), sp, ss, out.data_ptr(),
+                                          out.stride(0), num_heads, dk, dv, int(M >= 4 * seq_slots.numel()), _stream()),
+           "rl_gated_linear_scan")
+    _count()
+
+
+def gated_delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a_raw: torch.Tensor, b_raw: torch.Tensor, rate: torch.Tensor,
+                     dt_bias: torch.Tensor, unit_eps: float, q_scale: float, out: torch.Tensor, state: torch.Tensor,
+                     cu_seqlens: torch.Tensor, seq_slots: torch.Tensor, num_heads: int, heads_per_group: int, dk: int, dv: int) -> None:
+    """The gated delta rule for every head of every sequence of the step: q and k are made unit vectors a head (x /
+    sqrt(sum x^2 + unit_eps), q times q_scale); S = g S; u = beta (v - S^T k); S = S + k u^T; out = S^T q, with
+    g = exp(-exp(rate[h]) softplus(a_raw + dt_bias[h])) and beta = sigmoid(b_raw).  q, k [M, (H / heads_per_group) * dk], v
+    [M, H * dv], a_raw, b_raw [M, H] (views are fine), out float32 [M, H * dv]; the state (float [H, dv, dk] a slot) is
+    read from and left in ``state``."""
+    for t, name in ((q, "q"), (k, "k"), (v, "v"), (a_raw, "a_raw"), (b_raw, "b_raw")):
+        _need(t, name, q.dtype, contiguous=False)
+        assert t.stride(1) == 1
+    _need(out, "out", torch.float32); _need(rate, "rate", torch.float32); _need(dt_bias, "dt_bias", torch.float32)
+    _need(cu_seqlens, "cu_seqlens", torch.int32); _need(seq_slots, "seq_slots", torch.int32)
+    M = out.shape[0]
+    assert num_heads % heads_per_group == 0 and rate.numel() == num_heads and dt_bias.numel() == num_heads
+    assert out.shape == (M, num_heads * dv) and q.shape == (M, num_heads // heads_per_group * dk) and k.shape == q.shape
+    assert v.shape == (M, num_heads * dv) and a_raw.shape == (M, num_heads) and b_raw.shape == (M, num_heads)
+    sp, ss = _state_args(state)
+    assert state.shape[1] >= 4 * num_heads * dk * dv
+    _check(library().rl_gated_delta_scan(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), a_raw.data_ptr(),
+                                         a_raw.stride(0), b_raw.data_ptr(), b_raw.stride(0), _dt(q), rate.data_ptr(), dt_bias.data_ptr(),
+                                         float(unit_eps), float(q_scale), cu_seqlens.data_ptr(), seq_slots.data_ptr(), seq_slots.numel(),
+                                         sp, ss, out.data_ptr(), out.stride(0), num_heads, heads_per_group, dk, dv,
+                                         int(M >= 4 * seq_slots.numel()), _stream()), "rl_gated_delta_scan")
+    _count()
+
+
+class JoinTerm:
+    """A term of ``branch_join``: ``factor`` * y (float32 [M, d]); with ``norm`` (weight float32 [d], eps) the row is RMS-normed
+    first; with ``row`` (int32 [M * top]) y holds a mixture of experts' rows and the term is the sum of a token's choices,
+    times ``weights`` (float32 [M, top]; None: 1 each)."""
+    __slots__ = ("y", "factor", "norm_weight", "eps", "row", "weights", "top")
+
+    def __init__(self, y, factor=1.0, norm_weight=None, eps=0.0, row=None, weights=None, top=0):
+        self.y, self.factor, self.norm_weight, self.eps = y, float(factor), norm_weight, float(eps)
+        self.row, self.weights, self.top = row, weights, int(top)
+
+
+def branch_join(x: torch.Tensor, scale: float, terms: Sequence[JoinTerm], norm_weight: Optional[torch.Tensor] = None,
+                norm_bias: Optional[torch.Tensor] = None, norm_eps: float = 0.0, out: Optional[torch.Tensor] = None) -> None:
+    """x += scale * (the sum of at most four terms), x float32 [M, d]; with ``norm_weight`` (and ``norm_bias``) also
+    out = layer_norm(x), out [M, d] in its own dtype."""
+    _need(x, "x", torch.float32)
+    M, d = x.shape
+    n = len(terms)
+    ys, nws, rws, wts = ((_c_void_p * n)() for _ in range(4))
+    eps, fac, tops = (_c_float * n)(), (_c_float * n)(), (_c_int * n)()
+    for i, t in enumerate(terms):
+        _need(t.y, "y", torch.float32)
+        assert t.y.shape[1] == d
+        ys[i], fac[i], eps[i], tops[i] = t.y.data_ptr(), t.factor, t.eps, t.top
+        if t.row is not None:
+            _need(t.row, "row", torch.int32)
+            assert t.row.numel() == M * t.top and t.norm_weight is None
+            rws[i] = t.row.data_ptr()
+            if t.weights is not None:
+                _need(t.weights, "weights", torch.float32)
+                assert t.weights.shape == (M, t.top)
+                wts[i] = t.weights.data_ptr()
+        else:
+            assert t.y.shape == (M, d)
+        if t.norm_weight is not None:
+            _need(t.norm_weight, "norm_weight", torch.float32)
+            assert t.norm_weight.numel() == d
+            nws[i] = t.norm_weight.data_ptr()
+    if norm_weight is not None:
+        _need(norm_weight, "norm_weight", torch.float32); _need(out, "out")
+        assert norm_weight.numel() == d and out.shape == (M, d)
+        if norm_bias is not None:
+            _need(norm_bias, "norm_bias", torch.float32)
+            assert norm_bias.numel() == d
+    _check(library().rl_branch_join(x.data_ptr(), float(scale), n, ys, nws, eps, fac, rws, wts, tops, _ptr(norm_weight), _ptr(norm_bias),
+                                    float(norm_eps), _ptr(out), 0 if out is None else _dt(out), M, d, _stream()), "rl_branch_join")
+    _count()
+
+
 def norm_add(x: torch.Tensor, y0: torch.Tensor, s0: float, y1: Optional[torch.Tensor], s1: float, weight: torch.Tensor, eps: float,
              x_bf16: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
     """x += out_scale * rms_norm(s0 * y0 + s1 * y1) * weight, all float32 [M, d] (``y1`` may be ``None``); ``x_bf16``:
@@ -1424,8 +1561,9 @@ def num_sms() -> int:
     return _num_sms[dev]
 
 
-def attention_decode_supported(dtype: torch.dtype, num_heads: int, num_kv_heads: int, head_dim: int) -> bool:
-    return dtype == torch.bfloat16 and bool(library().rl_attention_decode_supported(num_heads, num_kv_heads, head_dim))
+def attention_decode_supported(dtype: torch.dtype, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: Optional[int] = None) -> bool:
+    return dtype == torch.bfloat16 and bool(library().rl_attention_decode_supported_shaped(num_heads, num_kv_heads, head_dim,
+                                                                                           head_dim if value_dim is None else value_dim))
 
 
 # One sequence alone: up to this many cached tokens its eight chunks run as one cluster that
@@ -1470,15 +1608,19 @@ def length_spread(kv_lens: Sequence[int]) -> int:
     return 2 if over <= FAR_SPREAD * n and max(kv_lens) * LONGEST_SHARE <= sum(kv_lens) else 3
 
 
-def decode_places(head_dim: int) -> int:
+def decode_places(head_dim: int, value_dim: Optional[int] = None) -> int:
     """CTAs of the decode kernel the GPU holds at once at this head size (296 at 128, 444 at 64)."""
-    n = int(library().rl_attention_decode_places(int(head_dim)))
+    n = int(library().rl_attention_decode_places_shaped(int(head_dim), int(head_dim if value_dim is None else value_dim)))
     if n <= 0:
         _check(n or -1, "rl_attention_decode_places")
     return n
 
 
-def decode_order_wanted(num_seqs: int, num_kv_heads: int, head_dim: int) -> bool:
+def _decode_ring_bytes(head_dim: int, value_dim: Optional[int]) -> int:
+    return int(library().rl_attention_decode_ring_bytes_shaped(int(head_dim), int(head_dim if value_dim is None else value_dim)))
+
+
+def decode_order_wanted(num_seqs: int, num_kv_heads: int, head_dim: int, value_dim: Optional[int] = None) -> bool:
     """Whole sequences that are more CTAs than the GPU holds at once (and keep 30 MB in flight
     among them) start in the order of their lengths, the longest first.  Sequences of 128 to 2,047
     tokens, in order against dealt chunks: head size 128, 40 sequences 36.4 / 38.6 us, 48: 39.1 /
@@ -1486,11 +1628,12 @@ def decode_order_wanted(num_seqs: int, num_kv_heads: int, head_dim: int) -> bool
     unsorted); head size 64, 96: 38.4 / 40.5, 128: 42.0 / 50.2, but 64 (24 MB in flight): 31.7 /
     30.4.  The order kernel takes up to 1,024 sequences."""
     ctas = num_seqs * num_kv_heads
-    ring = int(library().rl_attention_decode_ring_bytes(int(head_dim)))
-    return ctas > decode_places(head_dim) and ctas * ring >= 30_000_000 and num_seqs <= 1024
+    ring = _decode_ring_bytes(head_dim, value_dim)
+    return ctas > decode_places(head_dim, value_dim) and ctas * ring >= 30_000_000 and num_seqs <= 1024
 
 
-def decode_cluster_size(num_seqs: int, num_kv_heads: int, head_dim: int, long_context: bool, spread: int) -> int:
+def decode_cluster_size(num_seqs: int, num_kv_heads: int, head_dim: int, long_context: bool, spread: int,
+                        value_dim: Optional[int] = None) -> int:
     """How the decode attention cuts the sequences of a step: 8, 4 or 2 = so many equal chunks a
     sequence as one cluster; 1 = every sequence whole in one CTA a KV head; 0 = chunks dealt by
     length and a combining kernel.  One sequence alone: eight chunks up to the long-context mark.
@@ -1511,13 +1654,13 @@ def decode_cluster_size(num_seqs: int, num_kv_heads: int, head_dim: int, long_co
         return 8 if splits >= 8 and not long_context else 0
     if splits < 2:
         return 0
-    if decode_order_wanted(num_seqs, num_kv_heads, head_dim):
+    if decode_order_wanted(num_seqs, num_kv_heads, head_dim, value_dim):
         return 1 if spread <= 2 else 0
     if spread > 1:
         return 0
-    places, ctas = decode_places(head_dim), num_seqs * num_kv_heads
+    places, ctas = decode_places(head_dim, value_dim), num_seqs * num_kv_heads
     if ctas * 2 > places:
-        return 1 if ctas * int(library().rl_attention_decode_ring_bytes(int(head_dim))) >= 15_000_000 else 0
+        return 1 if ctas * _decode_ring_bytes(head_dim, value_dim) >= 15_000_000 else 0
     size = 8 if splits >= 8 else 4 if splits >= 4 else 2
     if spread == 1 and size != splits:
         return 0
@@ -1564,7 +1707,7 @@ def attention_decode(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
                      num_splits: Optional[int] = None, scratch: Optional[torch.Tensor] = None,
                      plan: Optional[torch.Tensor] = None, cluster: bool = False, sink: bool = False,
                      gate: Optional[torch.Tensor] = None, softcap: float = 0.0, keep_first: int = 0,
-                     gate_per_head: bool = False) -> None:
+                     gate_per_head: bool = False, value_dim: Optional[int] = None, sinks: Optional[torch.Tensor] = None) -> None:
     """One token per sequence over the bf16 cache, split over the context (tensor cores).
     q: [B, >= H*hd] bf16 (a view into the qkv buffer is fine); out: [B, H*hd] bf16.
     ``num_splits``: chunks per sequence; with a ``plan`` (from ``decode_plan`` with the
@@ -1573,7 +1716,9 @@ def attention_decode(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
     ``cluster`` (2, 4 or 8 splits, no plan): the chunks of a sequence run as a
     thread-block cluster and combine through shared memory - no scratch, one kernel.
     ``softcap`` > 0: a score s (scale included) becomes softcap * tanh(s / softcap); ``keep_first``: with a
-    window, positions [0, keep_first) stay visible."""
+    window, positions [0, keep_first) stay visible.  ``value_dim`` (64 or 128; default: head_dim): the width of a value head,
+    out is [B, H*value_dim].  ``sinks`` (float32 [H], with ``sink``): the extra term's score a head instead of 0."""
+    vd = head_dim if value_dim is None else value_dim
     _need(q, "q", torch.bfloat16, contiguous=False); _need(k_pool, "k_pool", torch.bfloat16)
     _need(v_pool, "v_pool", torch.bfloat16); _need(out, "out", torch.bfloat16)
     _need(page_table, "page_table", torch.int32); _need(seq_slots, "seq_slots", torch.int32)
@@ -1584,7 +1729,7 @@ def attention_decode(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
         num_splits = decode_splits(B, num_kv_heads)
     if cluster:
         assert plan is None and scratch is None and num_splits in (2, 4, 8)
-    need = 0 if cluster else decode_scratch_floats(B, num_heads, head_dim, num_splits)
+    need = 0 if cluster else decode_scratch_floats(B, num_heads, vd, num_splits)
     if num_splits > 1 and scratch is None and not cluster:
         scratch = torch.empty(need, dtype=torch.float32, device=q.device)
     if scratch is not None:
@@ -1594,12 +1739,13 @@ def attention_decode(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
         _need(plan, "plan", torch.int32)
         assert plan.numel() >= 4 * B * num_splits + 2 * B
     ldq = q.stride(0) if B > 1 else max(q.stride(0), num_heads * head_dim)
-    gptr, ldg = _gate_args(gate, B, num_heads if gate_per_head else num_heads * head_dim, 2)
-    _check(library().rl_attention_decode_headgate(
+    gptr, ldg = _gate_args(gate, B, num_heads if gate_per_head else num_heads * vd, 2)
+    _check(library().rl_attention_decode_wide(
         q.data_ptr(), ldq, k_pool.data_ptr(), v_pool.data_ptr(), page_table.data_ptr(), page_table.shape[1],
         seq_slots.data_ptr(), kv_lens.data_ptr(), out.data_ptr(), out.stride(0), _ptr(scratch), _ptr(plan), B,
         num_heads, num_kv_heads, head_dim, float(scale), int(window), int(num_splits), int(bool(sink)), gptr, ldg,
-        float(softcap or 0.0), int(keep_first or 0), int(bool(gate_per_head and gate is not None)), _stream()), "rl_attention_decode")
+        float(softcap or 0.0), int(keep_first or 0), int(bool(gate_per_head and gate is not None)), vd, _sinks(sinks, num_heads),
+        _stream()), "rl_attention_decode")
     _count(2 if num_splits > 1 and not cluster else 1)
 
 
@@ -1653,8 +1799,10 @@ def prefill_tile_order(q_lens, kv_lens, device) -> torch.Tensor:
     return torch.tensor([[b, t] for _, b, t in items], dtype=torch.int32).to(device, non_blocking=True)
 
 
-def attention_prefill_tc_supported(dtype: torch.dtype, num_heads: int, num_kv_heads: int, head_dim: int) -> bool:
-    return dtype == torch.bfloat16 and bool(library().rl_attention_prefill_tc_supported(num_heads, num_kv_heads, head_dim))
+def attention_prefill_tc_supported(dtype: torch.dtype, num_heads: int, num_kv_heads: int, head_dim: int,
+                                   value_dim: Optional[int] = None) -> bool:
+    return dtype == torch.bfloat16 and bool(library().rl_attention_prefill_tc_supported_shaped(num_heads, num_kv_heads, head_dim,
+                                                                                               head_dim if value_dim is None else value_dim))
 
 
 def attention_prefill_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_table: torch.Tensor,
@@ -1662,11 +1810,14 @@ def attention_prefill_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Te
                          out: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
                          window: int = 0, tile_order: Optional[torch.Tensor] = None, sink: bool = False,
                          gate: Optional[torch.Tensor] = None, softcap: float = 0.0, keep_first: int = 0, chunk: int = 0,
-                         gate_per_head: bool = False) -> None:
+                         gate_per_head: bool = False, value_dim: Optional[int] = None, sinks: Optional[torch.Tensor] = None) -> None:
     """The same as ``attention_prefill`` on tcgen05 tensor cores (head size 64 or 128).  ``chunk`` > 0 (instead of a
     window): a query at position p sees positions [p - p % chunk, p].  The cache
     pools must hold finite values everywhere (the cache zero-fills them when it allocates them).
-    ``tile_order``: what ``prefill_tile_order`` made for this step (the blocks then start heaviest first)."""
+    ``tile_order``: what ``prefill_tile_order`` made for this step (the blocks then start heaviest first).  ``value_dim``
+    (64 or 128; default: head_dim): the width of a value head.  ``sinks`` (float32 [H], with ``sink``): the extra term's score
+    a head instead of 0."""
+    vd = head_dim if value_dim is None else value_dim
     _need(q, "q", torch.bfloat16, contiguous=False); _need(k_pool, "k_pool", torch.bfloat16)
     _need(v_pool, "v_pool", torch.bfloat16); _need(out, "out", torch.bfloat16)
     _need(page_table, "page_table", torch.int32); _need(cu_seqlens, "cu_seqlens", torch.int32)
@@ -1679,13 +1830,14 @@ def attention_prefill_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Te
         _need(tile_order, "tile_order", torch.int32)
         assert tile_order.numel() == 2 * tiles
     ldq = q.stride(0) if q.shape[0] > 1 else max(q.stride(0), num_heads * head_dim)
-    gptr, ldg = _gate_args(gate, q.shape[0], num_heads, 2) if gate_per_head else _gate_args(gate, q.shape[0], num_heads * head_dim, 16)
-    _check(library().rl_attention_prefill_tc_headgate(
+    gptr, ldg = _gate_args(gate, q.shape[0], num_heads, 2) if gate_per_head else _gate_args(gate, q.shape[0], num_heads * vd, 16)
+    _check(library().rl_attention_prefill_tc_wide(
         q.data_ptr(), ldq, k_pool.data_ptr(), v_pool.data_ptr(), k_pool.shape[0], page_table.data_ptr(),
         page_table.shape[1], cu_seqlens.data_ptr(), seq_slots.data_ptr(), kv_lens.data_ptr(), B, tiles, q.shape[0],
         out.data_ptr(), out.stride(0), num_heads, num_kv_heads, head_dim, float(scale), int(window),
         _tc_error_word(q.device).data_ptr(), _ptr(tile_order), int(bool(sink)), gptr, ldg, float(softcap or 0.0),
-        int(keep_first or 0), int(chunk or 0), int(bool(gate_per_head and gate is not None)), _stream()), "rl_attention_prefill_tc")
+        int(keep_first or 0), int(chunk or 0), int(bool(gate_per_head and gate is not None)), vd, _sinks(sinks, num_heads),
+        _stream()), "rl_attention_prefill_tc")
     _count()
 
 
@@ -1739,12 +1891,12 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_
               step, out: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
               window: int = 0, value_dim: Optional[int] = None, sink: bool = False,
               gate: Optional[torch.Tensor] = None, softcap: float = 0.0, keep_first: int = 0, chunk: int = 0,
-              values_in_keys: bool = False, gate_per_head: bool = False) -> None:
+              values_in_keys: bool = False, gate_per_head: bool = False, sinks: Optional[torch.Tensor] = None) -> None:
     """Attention of the step's tokens over the cache; picks the kernel for the
     dtype and the shape of the step.  ``step`` carries positions, slots and
-    sequence boundaries (engine.step.StepState).  Value heads of another width than the
-    key heads (``value_dim``) run on the any-shape kernel; the tensor-core kernels take
-    one width for both.  ``sink``: one more term of score 0 in the softmax's denominator.
+    sequence boundaries (engine.step.StepState).  Key and value heads of 64 or 128 each (``value_dim``) run on the
+    tensor-core kernels, other widths on the any-shape kernel.  ``sink``: one more term of score 0 in the softmax's
+    denominator; ``sinks`` (float32 [H]): the same with a score a head.
     ``gate`` [M, H*vd]: the output is multiplied by sigmoid(gate) (``gate_per_head``: [M, H], one number a head).
     ``chunk`` > 0 instead of a window: a query sees the positions of its own block of ``chunk`` positions up to
     itself.  ``values_in_keys``: the values are the front part of the key rows (any-shape kernel)."""
@@ -1757,48 +1909,47 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_
         attention_shared_key(q, k_pool, page_table, step.cu_seqlens, step.seq_slots, step.kv_lens, step.q_lens, out,
                              num_heads, head_dim, head_dim if value_dim is None else value_dim, scale, window, gate=gate)
         return
-    vd_eff = head_dim if value_dim is None else value_dim
-    tc_head_gate = (gate_per_head and gate is not None and not values_in_keys and vd_eff == head_dim and q.dtype == torch.bfloat16
-                    and not chunk and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
-                    and (attention_decode_supported(q.dtype, num_heads, num_kv_heads, head_dim) if step.is_decode else
-                         attention_prefill_tc_supported(q.dtype, num_heads, num_kv_heads, head_dim)))
+    sink = bool(sink) or sinks is not None
+    decode_ok = step.is_decode and attention_decode_supported(q.dtype, num_heads, num_kv_heads, head_dim, value_dim)
+    prefill_ok = not step.is_decode and attention_prefill_tc_supported(q.dtype, num_heads, num_kv_heads, head_dim, value_dim)
+    tc_head_gate = (gate_per_head and gate is not None and not values_in_keys and q.dtype == torch.bfloat16
+                    and not chunk and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and (decode_ok or prefill_ok))
     if values_in_keys or (gate_per_head and not tc_head_gate):
         attention_simt(q, k_pool, v_pool, page_table, step.slot_of_token, step.positions, out,
                        num_heads, num_kv_heads, head_dim, scale, window, value_dim=value_dim, sink=sink, gate=gate,
                        softcap=softcap, keep_first=keep_first, chunk=chunk, values_in_keys=values_in_keys,
-                       gate_per_head=gate_per_head)
+                       gate_per_head=gate_per_head, sinks=sinks)
         return
     # the decode kernel and its plans take a chunked mask as a negative window
     dec_window = -int(chunk) if chunk else int(window)
     masked = bool(softcap or (keep_first and window) or chunk)
-    tc_prefill = (not step.is_decode and attention_prefill_tc_supported(q.dtype, num_heads, num_kv_heads, head_dim)
+    tc_prefill = (prefill_ok
                   and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
                   and (gate is None or gate_per_head or (gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0)))
-    if (value_dim is not None and value_dim != head_dim) or (masked and not tc_prefill and not (
-            step.is_decode and attention_decode_supported(q.dtype, num_heads, num_kv_heads, head_dim))):
-        # soft-capped scores, kept first tokens and chunked masks: the any-shape kernel, the decode kernel and the
-        # tcgen05 prompt kernel have them (the mma.sync prompt kernel does not)
+    if (masked or sinks is not None or (value_dim is not None and value_dim != head_dim)) and not tc_prefill and not decode_ok:
+        # soft-capped scores, kept first tokens, chunked masks, a sink's score a head and value heads of another width: the
+        # any-shape kernel, the decode kernel and the tcgen05 prompt kernel have them (the mma.sync prompt kernel does not)
         attention_simt(q, k_pool, v_pool, page_table, step.slot_of_token, step.positions, out,
                        num_heads, num_kv_heads, head_dim, scale, window, value_dim=value_dim, sink=sink, gate=gate,
-                       softcap=softcap, keep_first=keep_first, chunk=chunk)
+                       softcap=softcap, keep_first=keep_first, chunk=chunk, sinks=sinks)
         return
-    if step.is_decode and attention_decode_supported(q.dtype, num_heads, num_kv_heads, head_dim):
+    if decode_ok:
         splits = decode_splits(q.shape[0], num_kv_heads)
         cluster = decode_cluster_size(q.shape[0], num_kv_heads, head_dim, getattr(step, "long_context", False),
-                                      getattr(step, "length_spread", 3))
+                                      getattr(step, "length_spread", 3), value_dim)
         if cluster:
             # nothing to deal: equal chunks a sequence as one cluster, combined through shared memory,
             # or every sequence whole
             order = None
             derived = getattr(step, "derived", None)
-            if cluster == 1 and derived is not None and decode_order_wanted(q.shape[0], num_kv_heads, head_dim):
+            if cluster == 1 and derived is not None and decode_order_wanted(q.shape[0], num_kv_heads, head_dim, value_dim):
                 order = derived.get(("decode_order", dec_window))
                 if order is None:
                     order = derived[("decode_order", dec_window)] = decode_order(step.seq_slots, step.kv_lens, dec_window)
             attention_decode(q, k_pool, v_pool, page_table, step.seq_slots, step.kv_lens, out,
                              num_heads, num_kv_heads, head_dim, scale, dec_window, num_splits=cluster, plan=order,
                              cluster=cluster > 1, sink=sink, gate=gate, softcap=softcap, keep_first=keep_first,
-                             gate_per_head=gate_per_head)
+                             gate_per_head=gate_per_head, value_dim=value_dim, sinks=sinks)
             return
         plan = None
         derived = getattr(step, "derived", None)     # what layers of one step share
@@ -1809,7 +1960,7 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_
                 plan = derived[key] = decode_plan(step.seq_slots, step.kv_lens, dec_window, splits)
         attention_decode(q, k_pool, v_pool, page_table, step.seq_slots, step.kv_lens, out,
                          num_heads, num_kv_heads, head_dim, scale, dec_window, num_splits=splits, plan=plan, sink=sink, gate=gate,
-                         softcap=softcap, keep_first=keep_first, gate_per_head=gate_per_head)
+                         softcap=softcap, keep_first=keep_first, gate_per_head=gate_per_head, value_dim=value_dim, sinks=sinks)
         return
     if tc_prefill:
         order = None
@@ -1820,7 +1971,8 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_
                 order = derived["prefill_tile_order"] = prefill_tile_order(step.q_lens, step.kv_lens_host, q.device)
         attention_prefill_tc(q, k_pool, v_pool, page_table, step.cu_seqlens, step.seq_slots, step.kv_lens,
                              step.q_lens, out, num_heads, num_kv_heads, head_dim, scale, window, tile_order=order,
-                             sink=sink, gate=gate, softcap=softcap, keep_first=keep_first, chunk=chunk, gate_per_head=gate_per_head)
+                             sink=sink, gate=gate, softcap=softcap, keep_first=keep_first, chunk=chunk, gate_per_head=gate_per_head,
+                             value_dim=value_dim, sinks=sinks)
         return
     if not chunk and not step.is_decode and attention_prefill_supported(q.dtype, num_heads, num_kv_heads, head_dim) \
             and (gate is None or (gate.data_ptr() % 4 == 0 and gate.stride(0) % 2 == 0)):

@@ -191,6 +191,8 @@ class DecoderModel:
                 # a norm is not started across an injection: the stream changes between the two layers
                 want = nxt.first_norm_request(x.shape[0]) if nxt is not None and nxt.folds_norms \
                     and (pos + 1) not in self.injections else None
+                if want is not None and not isinstance(want, block.norm_requests):
+                    want = None          # a norm this block cannot start
                 pending = block.forward(x, step, view, pending=pending, next_norm=want)
             else:
                 block.forward(x, step, view)

@@ -82,7 +82,7 @@ def eligible(model, cache) -> bool:
         if type(b.mixer_norm) is not RMSNorm or type(b.feed_forward_norm) is not RMSNorm or not isinstance(b.mixer.position, RotaryEmbedding):
             return False
         a, f = b.mixer, b.feed_forward
-        if a.sink or a.gated or getattr(a, "value_mix", None) or f.activation != "silu":
+        if a.sink or a.gated or getattr(a, "value_mix", None) or a.shared_keys or f.activation != "silu":
             return False
         if not (f.interleaved and _matrix_ok(a.wqkv) and _matrix_ok(a.wo) and _matrix_ok(f.wgu) and _matrix_ok(f.wdown)):
             return False

@@ -20,7 +20,9 @@ before rotation and norm, with no value projection (``value_from_key``); an outp
 instead of one an element (``gate_per_head``: Wg has H rows); values blended with another layer's values of the same
 token before they are cached, v <- (1 - lam) v + lam v_other (``value_mix`` = {"key": k, "role": "source" or "blend"}:
 the "source" layer of a key leaves its values of the step's tokens for the "blend" layers that run after it; lam is
-the learned scalar ``names["vmix"]``).  Here Wq, Wk, Wv are one matrix [(H + 2G) hd x d] so that one product
+the learned scalar ``names["vmix"]``); a sink whose score is a learned number a head (``names["sink"]``: p_j = e^{s_j} /
+(e^{sink_h} + sum_t e^{s_t})); no keys and values of its own (``shared_keys``: the layer reads the entry of the layer that
+``LayerSpec.cache_from`` names, as that one's cache holds it, with queries of its own).  Here Wq, Wk, Wv are one matrix [(H + 2G) hd x d] so that one product
 serves all three, rotation and cache write are one kernel, and all tokens of the
 step (several sequences, prompt or single tokens) run together.
 """
@@ -47,7 +49,8 @@ class GQAttention(Mixer):
                  scale: Optional[float] = None, sink: bool = False, conv_taps: int = 0,
                  qk_norm_eps: Optional[float] = None, softcap: Optional[float] = None, keep_first: int = 0,
                  bias_o: Optional[bool] = None, chunk: Optional[int] = None, unit_qk_eps: Optional[float] = None,
-                 value_from_key: bool = False, gate_per_head: bool = False, value_mix: Optional[Dict[str, str]] = None):
+                 value_from_key: bool = False, gate_per_head: bool = False, value_mix: Optional[Dict[str, str]] = None,
+                 shared_keys: bool = False):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads are no multiple of {num_kv_heads} KV heads")
         if head_dim % 2 or not (0 < head_dim <= 256):
@@ -64,7 +67,13 @@ class GQAttention(Mixer):
         self.window = window
         self.names = names
         self.scale = 1.0 / math.sqrt(head_dim) if scale is None else float(scale)     # src/model.rs:7239
-        self.sink = bool(sink)
+        self.sink = bool(sink) or "sink" in names
+        self.sinks = None                  # the sink's score a head, where it is learned
+        self.shared_keys = bool(shared_keys)
+        if self.shared_keys and (bias or conv_taps or "q_norm" in names or "k_norm" in names or value_from_key or unit_qk_eps is not None
+                                 or value_mix is not None):
+            raise ValueError("a layer on another layer's keys together with biases, a convolution, head norms, unit-size heads or blended "
+                             "values is not built")
         self.gated = "g" in names          # an output gate: its rows ride behind q, k, v in the one product
         self.position = build_part("position", position, runtime)
         self.wqkv = self.wo = self.bqkv = self.bo = None
@@ -112,8 +121,10 @@ class GQAttention(Mixer):
     def param_specs(self) -> Dict[str, ParamSpec]:
         d, H, G, hd, vd, n = self.d, self.H, self.G, self.hd, self.vd, self.names
         sfx = n.get("suffix", ".weight")     # what follows a projection's name in the checkpoint
-        qkv = (ParamSource(n["q"] + sfx, (H * hd, d)), ParamSource(n["k"] + sfx, (G * hd, d)))
-        if not self.value_from_key:
+        qkv = (ParamSource(n["q"] + sfx, (H * hd, d)),)
+        if not self.shared_keys:
+            qkv += (ParamSource(n["k"] + sfx, (G * hd, d)),)
+        if not self.value_from_key and not self.shared_keys:
             qkv += (ParamSource(n["v"] + sfx, (G * vd, d)),)
         if self.gated:
             qkv += (ParamSource(n["g"] + sfx, (self.gate_rows, d)),)
@@ -131,6 +142,8 @@ class GQAttention(Mixer):
                                          ParamSource(n["v"] + csfx, (G * vd, t))), role="vector")
         if self.value_mix is not None and self.value_mix["role"] == "blend":
             specs["vmix"] = ParamSpec((ParamSource(n["vmix"], ()),), role="vector", init="zeros")
+        if "sink" in n:
+            specs["sinks"] = ParamSpec((ParamSource(n["sink"], (H,)),), role="vector", init="zeros")
         if "q_norm" in n:
             specs["q_norm_w"] = ParamSpec((ParamSource(n["q_norm"], (hd,)),), role="vector", init="ones")
         if "k_norm" in n:
@@ -167,7 +180,9 @@ class GQAttention(Mixer):
         H, G, hd, vd = self.H, self.G, self.hd, self.vd
         M = xn.shape[0]
         dt = xn.dtype
-        n_qkv = (H + G) * hd + (0 if self.value_from_key else G * vd)
+        n_qkv = H * hd if self.shared_keys else (H + G) * hd + (0 if self.value_from_key else G * vd)
+        if self.shared_keys and cache.writes:
+            raise K.KernelError("a layer without keys and values of its own was given a cache entry of its own to read")
         width = n_qkv + self.gate_rows
         # rows a multiple of 8 elements apart (the tensor-core attention kernels read queries by 16-byte pieces): a gate of
         # one number a head can leave the row's length odd
@@ -187,7 +202,14 @@ class GQAttention(Mixer):
         magnitude = getattr(pos, "magnitude", 1.0)      # a position kind of its own need not know the attribute
         prepared = self.conv_taps or self.qk_norm or magnitude != 1.0
         q = qkv
-        if self.value_from_key or self.unit_qk_eps is not None:
+        if self.shared_keys:
+            # queries alone: the keys and values are in the other layer's entry already
+            linear(xn, self.wqkv, qkv, OUT_SAME)
+            if magnitude != 1.0:
+                raise K.KernelError("a magnitude on the rotation of queries alone is not built")
+            K.rope_kv_write(qkv, step.positions, step.slot_of_token, group.page_table, pos.inv_freq, H, 0, hd, pos.rotary_dim,
+                            pos.interleaved, None, None, value_dim=vd)
+        elif self.value_from_key or self.unit_qk_eps is not None:
             # rotation first, then heads of unit size; the keys as projected are the values: one kernel behind the product
             linear(xn, self.wqkv, qkv, OUT_SAME, self.bqkv)
             if not self.value_from_key:
@@ -225,6 +247,6 @@ class GQAttention(Mixer):
             step.derived[("values", self.value_mix["key"])] = qkv[:, (H + G) * hd:(H + G) * hd + G * vd]
         attn = torch.empty((M, H * vd), dtype=dt, device=xn.device)
         K.attention(q, k_pool, v_pool, group.page_table, step, attn, H, G, hd, self.scale,
-                    self.window or 0, value_dim=vd, sink=self.sink, gate=qkv[:, n_qkv:] if self.gated else None,
+                    self.window or 0, value_dim=vd, sink=self.sink, sinks=self.sinks, gate=qkv[:, n_qkv:] if self.gated else None,
                     softcap=self.softcap, keep_first=self.keep_first, chunk=self.chunk or 0, gate_per_head=self.gate_per_head)
         return linear(attn, self.wo, residual, _out_mode, self.bo, then_norm=then_norm)

@@ -78,6 +78,24 @@ class NormedInput:
 
 
 @dataclass(frozen=True)
+class LayerNormRequest:
+    """What whoever adds a layer's outputs into the stream needs to make the next layer's input on the way:
+    y = (x - mean) / sqrt(variance + eps) * weight + bias."""
+    weight: torch.Tensor          # [d] float32
+    bias: Optional[torch.Tensor]  # [d] float32 or None
+    eps: float
+
+
+@dataclass
+class NormedTerm:
+    """A mixer's output that is to be RMS-normed over the whole width before it joins the stream, the norm still to be
+    taken: y / sqrt(mean(y^2) + eps) * weight.  For whoever adds it into the stream."""
+    y: torch.Tensor               # float32 [M, d]
+    weight: torch.Tensor          # [d] float32
+    eps: float
+
+
+@dataclass(frozen=True)
 class Runtime:
     """Where and in which precision a model runs."""
     device: torch.device
@@ -151,6 +169,9 @@ class Block(Part):
     # True for a block whose ``forward`` takes ``pending`` and ``next_norm``; a block that
     # leaves this False is called as ``forward(x, step, cache)``.
     folds_norms: bool = False
+    # the kinds of request its ``next_norm`` may be; a request of another kind (the next block's norm is of a kind this
+    # block cannot start) is not handed to it
+    norm_requests = (NormRequest,)
 
     def forward(self, x: torch.Tensor, step, cache, pending=None, next_norm=None):
         """Updates the residual x in place.  ``pending``: the block's first norm of x,

@@ -5,7 +5,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import Block, FeedForward, Mixer, Norm, Runtime
+from .base import Block, FeedForward, LayerNormRequest, Mixer, Norm, NormedTerm, Runtime
 from .registry import register_block
 
 
@@ -88,6 +88,68 @@ class ParallelPreNormBlock(Block):
         self.mixer.forward(h1, x, step, cache)
         self.feed_forward.forward(h2, x, step)
         return None
+
+
+@register_block("parallel_shared_norm")
+class ParallelSharedNormBlock(Block):
+    """A layer with one norm that both sublayers read, joined together with a constant:
+
+        h = norm(x);   x += residual_scale * (mixer(h) + feed_forward(h))
+
+    Where the norm is a layer norm, one kernel adds a layer's outputs into the stream - a mixer's (normed first where it
+    returns ``NormedTerm``s), the feed-forward's, the experts' rows summed on the way - and takes the next layer's norm
+    of the result: between two layers the stream is read and written once."""
+
+    def __init__(self, runtime: Runtime, mixer: Mixer, mixer_norm: Norm, feed_forward: FeedForward, feed_forward_norm: Norm,
+                 residual_scale: float = 1.0):
+        self.runtime = runtime
+        self.residual_scale = float(residual_scale)
+        self.mixer, self.mixer_norm = mixer, mixer_norm
+        self.feed_forward, self.feed_forward_norm = feed_forward, feed_forward_norm
+        if type(feed_forward_norm).__name__ != "NoNorm":
+            raise ValueError("a parallel_shared_norm block has one norm, the mixer's: the feed-forward's must be of kind 'none'")
+
+    def sub_parts(self):
+        return {"mixer": self.mixer, "mixer_norm": self.mixer_norm,
+                "feed_forward": self.feed_forward, "feed_forward_norm": self.feed_forward_norm}
+
+    folds_norms = True
+    norm_requests = (LayerNormRequest,)
+
+    def first_norm_request(self, num_tokens: int):
+        return self.mixer_norm.layer_request() if hasattr(self.mixer_norm, "layer_request") else None
+
+    @staticmethod
+    def _terms(part, h, *args, **ok):
+        """A sublayer's output as terms of its own; a part that can only add into the stream adds into zeros."""
+        if hasattr(part, "forward_out"):
+            return part.forward_out(h, *args, **ok)
+        y = torch.zeros(h.shape, dtype=torch.float32, device=h.device)
+        part.forward(h, y, *args)
+        return [(y, 1.0)]
+
+    def forward(self, x: torch.Tensor, step, cache, pending=None, next_norm=None):
+        from .. import kernels as K
+        from .moe import ExpertRows
+        h = pending if pending is not None else self.mixer_norm.forward(x, self.runtime.compute_dtype)
+        terms = self._terms(self.mixer, h, step, cache, **({"normed_ok": True} if getattr(self.mixer, "offers_normed", False) else {}))
+        ff = self.feed_forward
+        if not getattr(ff, "absent", False):
+            terms = terms + self._terms(ff, h, step, **({"rows_ok": True} if getattr(ff, "offers_rows", False) else {}))
+        joins = []
+        for y, f in terms:
+            if isinstance(y, NormedTerm):
+                joins.append(K.JoinTerm(y.y, f, norm_weight=y.weight, eps=y.eps))
+            elif isinstance(y, ExpertRows):
+                joins.append(K.JoinTerm(y.rows, f, row=y.row, weights=y.weights, top=y.top))
+            else:
+                joins.append(K.JoinTerm(y, f))
+        if next_norm is None:
+            K.branch_join(x, self.residual_scale, joins)
+            return None
+        out = torch.empty(x.shape, dtype=self.runtime.compute_dtype, device=x.device)
+        K.branch_join(x, self.residual_scale, joins, next_norm.weight, next_norm.bias, next_norm.eps, out)
+        return out
 
 
 @register_block("post_norm")

@@ -35,7 +35,8 @@ class ExpertRows:
     ``rows`` and counts ``weights[m, c]``.  For whoever sums them on the way into the residual."""
     rows: torch.Tensor            # float32 [*, d]
     row: torch.Tensor             # int32 [M * top]
-    weights: torch.Tensor         # float32 [M, top]
+    weights: Optional[torch.Tensor]      # float32 [M, top]; None: 1 each (the weights went into the experts' inputs)
+    top: int
 
 
 @register_feed_forward("moe_mlp")
@@ -43,7 +44,7 @@ class MoEMLP(FeedForward):
     def __init__(self, runtime: Runtime, hidden_size: int, expert_size: int, num_experts: int, top: int,
                  names: Dict[str, str], router_bias: bool = True, shared: Optional[PartSpec] = None,
                  scoring: str = "softmax", groups: int = 1, keep_groups: int = 1, weight_scale: float = 1.0,
-                 activation: str = "silu", limit: Optional[float] = None, alpha: Optional[float] = None):
+                 activation: str = "silu", limit: Optional[float] = None, alpha: Optional[float] = None, weigh: str = "output"):
         """``names``: "router" (the router's matrix; its bias is that name + ``names["bias_suffix"]``),
         "expert" (a format string with ``{e}`` for the expert's number, giving the prefix of its
         "gate", "up" and "down" tensors), "suffix" (what follows a projection's name)."""
@@ -61,6 +62,10 @@ class MoEMLP(FeedForward):
         # largest choice scores); the weights are the chosen experts' s, not renormalised
         # ``weight_scale``: a constant on every weight (scores other than "softmax").  ``activation`` "clamped_sigmoid":
         # an expert is Wdown (g sigmoid(alpha g) (u + 1)) with g = min(Wgate x, limit), u = clamp(Wup x, -limit, limit)
+        # ``weigh`` "input": a weight multiplies what its expert reads, sum_c expert_c(w_c x), instead of what it returns
+        if weigh not in ("output", "input"):
+            raise ValueError(f"weigh {weigh!r} is not known; known: 'output', 'input'")
+        self.weigh_input = weigh == "input"
         if activation not in ("silu", "clamped_sigmoid"):
             raise ValueError(f"activation {activation!r} is not known; known: 'silu', 'clamped_sigmoid'")
         if activation == "clamped_sigmoid" and (limit is None or alpha is None or not limit > 0):
@@ -140,8 +145,8 @@ class MoEMLP(FeedForward):
             wgu, wd = self.wgu.view(self.E, self.F, 2, self.d), self.wdown.view(self.E, self.d, self.F)
             if self.use_grouped and K.moe_experts_grouped_supported(xn, wgu, wd):
                 ids, weights = self.route(xn)
-                rows, row = K.moe_experts_grouped(xn, wgu, wd, ids, weights, None, act=self.act)
-                return [(ExpertRows(rows, row, weights), 1.0)]
+                rows, row = K.moe_experts_grouped(xn, wgu, wd, ids, weights, None, act=self.act, weigh_input=self.weigh_input)
+                return [(ExpertRows(rows, row, None if self.weigh_input else weights, self.top), 1.0)]
         y = torch.zeros((xn.shape[0], self.d), dtype=torch.float32, device=xn.device)
         self.forward(xn, y, step)
         return [(y, 1.0)]
@@ -178,11 +183,12 @@ class MoEMLP(FeedForward):
         if self.interleaved:
             wgu = self.wgu.view(self.E, self.F, 2, self.d)
             if self.use_grouped and K.moe_experts_grouped_supported(xn, wgu, wd):
-                K.moe_experts_grouped(xn, wgu, wd, ids, weights, residual, act=self.act)
+                K.moe_experts_grouped(xn, wgu, wd, ids, weights, residual, act=self.act, weigh_input=self.weigh_input)
             else:
-                K.moe_experts(xn, wgu, wd, ids, weights, residual, interleaved=True, act=self.act)
+                K.moe_experts(xn, wgu, wd, ids, weights, residual, interleaved=True, act=self.act, weigh_input=self.weigh_input)
         else:
-            K.moe_experts(xn, self.wgu.view(self.E, 2, self.F, self.d), wd, ids, weights, residual, act=self.act)
+            K.moe_experts(xn, self.wgu.view(self.E, 2, self.F, self.d), wd, ids, weights, residual, act=self.act,
+                          weigh_input=self.weigh_input)
         if self.shared_gated and self.shared is not None:
             (y, _), = self.shared.forward_out(xn, step)
             K.row_gate_add(residual, y, xn, self.shared_gate)

@@ -16,7 +16,7 @@ import torch
 
 from .. import kernels as K
 from ..config.spec import ParamSource, ParamSpec
-from .base import Norm, NormRequest, Runtime
+from .base import LayerNormRequest, Norm, NormRequest, Runtime
 from .registry import register_norm
 
 
@@ -54,27 +54,38 @@ class RMSNorm(Norm):
 @register_norm("layer_norm")
 class LayerNorm(Norm):
     """y = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * w: the mean is taken off, the variance is the mean of
-    the squared deviations, there is a weight and no bias; all in 32-bit.  ``forward_with`` norms the same rows with
-    a second norm of this kind in the same kernel (a layer whose two sublayers read norms of one stream)."""
+    the squared deviations, there is a weight and, where ``bias_name`` names one, a bias (+ b); all in 32-bit.
+    ``forward_with`` norms the same rows with a second norm of this kind in the same kernel (a layer whose two sublayers
+    read norms of one stream; neither with a bias)."""
 
-    def __init__(self, runtime: Runtime, size: int, eps: float, name: str):
+    def __init__(self, runtime: Runtime, size: int, eps: float, name: str, bias_name: Optional[str] = None):
         self.runtime = runtime
         self.size = size
         self.eps = float(eps)
         self.name = name
+        self.bias_name = bias_name
         self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
-        return {"weight": ParamSpec((ParamSource(self.name, (self.size,)),), role="vector", init="ones")}
+        specs = {"weight": ParamSpec((ParamSource(self.name, (self.size,)),), role="vector", init="ones")}
+        if self.bias_name is not None:
+            specs["bias"] = ParamSpec((ParamSource(self.bias_name, (self.size,)),), role="vector", init="zeros")
+        return specs
 
     def forward(self, x: torch.Tensor, out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         n = x.shape[0] if rows is None else rows.numel()
         out = torch.empty((n, self.size), dtype=out_dtype, device=x.device)
-        K.layer_norm(x, self.weight, out, self.eps, rows)
+        K.layer_norm(x, self.weight, out, self.eps, rows, bias=self.bias)
         return out
 
+    def layer_request(self) -> LayerNormRequest:
+        """What a kernel that finishes a row of the stream needs to take this norm of it on the way."""
+        return LayerNormRequest(self.weight, self.bias, self.eps)
+
     def pairs_with(self, other: Norm) -> bool:
-        return isinstance(other, LayerNorm) and other.size == self.size and other.eps == self.eps
+        return (isinstance(other, LayerNorm) and other.size == self.size and other.eps == self.eps
+                and self.bias_name is None and other.bias_name is None)
 
     def forward_with(self, other: "LayerNorm", x: torch.Tensor, out_dtype: torch.dtype):
         out = torch.empty((2, x.shape[0], self.size), dtype=out_dtype, device=x.device)

@@ -1,7 +1,7 @@
 """Mixers that carry a state from token to token instead of caching keys and values.
 
 The first two are the same recurrence, S_t = a_t S_{t-1} + b_t k_t v_t^T with the output o_t = S_t^T q_t (csrc/linear_scan.cu),
-with different decays and different parts around it:
+with different decays and different parts around it (two more, further below, have kernels of their own, csrc/state_scan.cu):
 
 ``decay_linear_attention``
     q, k, v = silu(W h); a head's decay is a constant of the model, b = 1; the concatenated heads are RMS-normed
@@ -24,13 +24,18 @@ import torch
 from .. import kernels as K
 from ..cache.sequence_cache import StateNeed
 from ..config.spec import ParamSource, ParamSpec
-from .base import Mixer, Runtime
+from .base import Mixer, NormedTerm, Runtime
 from .linear import OUT_ADD_F32, OUT_F32, OUT_SAME, linear
 from .registry import register_mixer
 
 
 def _aligned(nbytes: int) -> int:
     return -(-nbytes // 256) * 256
+
+
+def _padded_rows(rows: int, width: int, dtype, device) -> torch.Tensor:
+    """An uninitialised [rows, width] whose rows are a multiple of 8 elements apart (16-byte pieces a row for its readers)."""
+    return torch.empty((rows, -(-width // 8) * 8), dtype=dtype, device=device)[:, :width]
 
 
 class _StateMixer(Mixer):
@@ -342,17 +347,164 @@ class GatedLinearRecurrence(_StateMixer):
         linear(o, self.wo, residual, _out_mode)
 
 
+@register_mixer("gated_linear_attention")
+class GatedLinearAttention(_StateMixer):
+    """Linear attention with a learned decay a key channel (Yang et al., "Gated Linear Attention Transformers with
+    Hardware-Efficient Training"):
+
+        q = head_dim^-1/2 W_q h,  k = W_k h,  v = W_v h;    a = sigmoid(W_2 (W_1 h) + c)^(1/tau), a value a head and key channel
+        S_t = diag(a_t) S_{t-1} + k_t v_t^T,   o_t = S_t^T q_t;    out = W_o (o / rms(o, per head) * norm * silu(W_g h))
+
+    with one norm weight for all heads.  The per-sequence state is the heads' matrices, float32, zero for a fresh sequence.
+    The decays (from the second projection's 32-bit sums on), the state, the sums and the head norm are 32-bit in every run;
+    the projections take the compute dtype.  q, k, v, the gate and the first of the decay's two projections are one product."""
+
+    def __init__(self, runtime: Runtime, hidden_size: int, num_heads: int, head_dim: int, value_dim: int, decay_rank: int, tau: float,
+                 norm_eps: float, names: Dict[str, str]):
+        """``names``: "q", "k", "v", "g", "o" (matrices), "a1", "a2" (the decay's projections; the second's bias: +
+        ``names["bias_suffix"]``), "norm" (weight [value_dim] behind the head norm), "suffix"."""
+        if not (0 < head_dim <= 256) or value_dim <= 0 or num_heads <= 0 or decay_rank <= 0:
+            raise ValueError(f"head_dim {head_dim} must lie in (0, 256], value_dim {value_dim}, heads {num_heads} and decay_rank {decay_rank} be positive")
+        if not tau > 0:
+            raise ValueError(f"tau {tau} must be > 0")
+        self.runtime = runtime
+        self.d, self.H, self.dk, self.dv, self.rank = hidden_size, num_heads, head_dim, value_dim, int(decay_rank)
+        self.tau, self.eps, self.names = float(tau), float(norm_eps), names
+        self.w_in = self.a2 = self.a2_b = self.norm_w = self.wo = None
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        d, H, dk, dv, n = self.d, self.H, self.dk, self.dv, self.names
+        sfx = n.get("suffix", ".weight")
+        return {
+            "w_in": ParamSpec((ParamSource(n["q"] + sfx, (H * dk, d)), ParamSource(n["k"] + sfx, (H * dk, d)),
+                               ParamSource(n["v"] + sfx, (H * dv, d)), ParamSource(n["g"] + sfx, (H * dv, d)),
+                               ParamSource(n["a1"] + sfx, (self.rank, d)))),
+            "a2": ParamSpec((ParamSource(n["a2"] + sfx, (H * dk, self.rank)),)),
+            "a2_b": ParamSpec((ParamSource(n["a2"] + n.get("bias_suffix", ".bias"), (H * dk,)),), role="vector", init="normal"),
+            "norm_w": ParamSpec((ParamSource(n["norm"], (dv,)),), role="vector", init="ones"),
+            "wo": ParamSpec((ParamSource(n["o"] + sfx, (d, H * dv)),)),
+        }
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        if "norm_w" in tensors:
+            tensors = dict(tensors, norm_w=tensors["norm_w"].repeat(self.H))
+        super().bind(tensors)
+
+    def state_need(self) -> StateNeed:
+        return StateNeed(4 * self.H * self.dk * self.dv)
+
+    def forward(self, xn, residual: torch.Tensor, step, cache, _out_mode=OUT_ADD_F32):
+        H, dk, dv = self.H, self.dk, self.dv
+        M, dt, dev = xn.shape[0], xn.dtype, xn.device
+        state = self._state(cache)
+        nk, nv = H * dk, H * dv
+        proj = _padded_rows(M, 2 * nk + 2 * nv + self.rank, dt, dev)
+        linear(xn, self.w_in, proj, OUT_SAME)
+        z = torch.empty((M, nk), dtype=torch.float32, device=dev)
+        linear(proj[:, 2 * nk + 2 * nv:], self.a2, z, OUT_F32, self.a2_b)
+        o = torch.empty((M, nv), dtype=torch.float32, device=dev)
+        K.gated_linear_scan(proj[:, :nk], proj[:, nk:2 * nk], proj[:, 2 * nk:2 * nk + nv], z, self.tau, dk ** -0.5, o, state,
+                            step.cu_seqlens, step.seq_slots, H, dk, dv)
+        on = torch.empty((M, nv), dtype=dt, device=dev)
+        K.gated_norm(o, proj[:, 2 * nk + nv:2 * nk + 2 * nv], self.norm_w, self.eps, on, groups=H, gate_act="silu", gate_first=False)
+        linear(on, self.wo, residual, _out_mode)
+
+
+@register_mixer("gated_delta_rule")
+class GatedDeltaRule(_StateMixer):
+    """A matrix state a head that is corrected towards each token's value instead of added to, with a decay a head (Yang et al.,
+    "Gated Delta Networks: Improving Mamba2 with Delta Rule"):
+
+        q, k, v = silu(causal filter over time of W h), a filter a channel; q, k divided by sqrt(sum of squares + unit_eps) a
+        head, q times head_dim^-1/2;   beta = sigmoid(W_b h),  g = exp(-exp(A_log) softplus(W_a h + dt_bias)), a number a head
+        S = g S;  u = beta (v - S^T k);  S = S + k u^T;  o = S^T q;      out = W_o (o / rms(o, per head) * norm * silu(W_g h))
+
+    Query/key heads may be fewer than value heads (head h reads q/k head h // (heads / kv_heads)); one norm weight for all
+    heads.  The per-sequence state is the filters' last taps - 1 inputs and the heads' matrices, float32, zero for a fresh
+    sequence.  Unit vectors, step sizes, decays, the state, the sums and the head norm are 32-bit in every run; projections and
+    filters' outputs take the compute dtype.  All projections of h are one product."""
+
+    def __init__(self, runtime: Runtime, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, conv_taps: int,
+                 norm_eps: float, names: Dict[str, str], unit_eps: float = 1e-6):
+        """``names``: "q", "k", "v", "g", "a", "b", "o" (matrices; the first three with filters [channels, taps], +
+        ``names["conv_suffix"]``), "A_log", "dt_bias" (a value a head), "norm" (weight [value_dim]), "suffix"."""
+        if num_kv_heads <= 0 or num_heads % num_kv_heads:
+            raise ValueError(f"{num_heads} heads are no multiple of {num_kv_heads} query/key heads")
+        if not (0 < head_dim <= 256) or value_dim <= 0:
+            raise ValueError(f"head_dim {head_dim} must lie in (0, 256] and value_dim {value_dim} be positive")
+        if not (1 <= conv_taps <= 8):
+            raise ValueError(f"conv_taps {conv_taps} outside [1, 8]")
+        self.runtime = runtime
+        self.d, self.H, self.G, self.dk, self.dv = hidden_size, num_heads, num_kv_heads, head_dim, value_dim
+        self.taps, self.eps, self.unit_eps, self.names = int(conv_taps), float(norm_eps), float(unit_eps), names
+        self.channels = 2 * self.G * self.dk + self.H * self.dv
+        self._conv_bytes = _aligned(4 * (self.taps - 1) * self.channels)
+        self.w_in = self.conv_w = self.a_log = self.dt_bias = self.norm_w = self.wo = None
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        d, H, G, dk, dv, n = self.d, self.H, self.G, self.dk, self.dv, self.names
+        sfx, csfx = n.get("suffix", ".weight"), n.get("conv_suffix", ".conv")
+        rows = (("q", G * dk), ("k", G * dk), ("v", H * dv))
+        return {
+            "w_in": ParamSpec(tuple(ParamSource(n[key] + sfx, (r, d)) for key, r in rows + (("g", H * dv), ("a", H), ("b", H)))),
+            "conv_w": ParamSpec(tuple(ParamSource(n[key] + csfx, (r, self.taps)) for key, r in rows), role="vector", init="normal"),
+            "a_log": ParamSpec((ParamSource(n["A_log"], (H,)),), role="vector", init="zeros"),
+            "dt_bias": ParamSpec((ParamSource(n["dt_bias"], (H,)),), role="vector", init="zeros"),
+            "norm_w": ParamSpec((ParamSource(n["norm"], (dv,)),), role="vector", init="ones"),
+            "wo": ParamSpec((ParamSource(n["o"] + sfx, (d, H * dv)),)),
+        }
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        if "norm_w" in tensors:
+            tensors = dict(tensors, norm_w=tensors["norm_w"].repeat(self.H))
+        super().bind(tensors)
+
+    def state_need(self) -> StateNeed:
+        # the filters' last taps - 1 inputs, then the heads' matrix states
+        return StateNeed(self._conv_bytes + 4 * self.H * self.dk * self.dv)
+
+    def forward(self, xn, residual: torch.Tensor, step, cache, _out_mode=OUT_ADD_F32):
+        H, G, dk, dv, C = self.H, self.G, self.dk, self.dv, self.channels
+        M, dt, dev = xn.shape[0], xn.dtype, xn.device
+        state = self._state(cache)
+        scan_state = state[:, self._conv_bytes:]
+        conv_state = state[:, :self._conv_bytes] if self.taps > 1 else state      # one tap: nothing is kept or read
+        nk, nv = G * dk, H * dv
+        proj = _padded_rows(M, C + nv + 2 * H, dt, dev)
+        linear(xn, self.w_in, proj, OUT_SAME)
+        u = proj[:, :C]
+        c = torch.empty((M, C), dtype=dt, device=dev)
+        if step.is_decode and self.taps > 1:
+            K.short_conv_step(u, self.conv_w, None, True, step.seq_slots, conv_state, c)
+        else:
+            K.short_conv(u, self.conv_w, None, True, step.slot_of_token, conv_state, c)
+            K.short_conv_state(u, self.taps, step.cu_seqlens, step.seq_slots, conv_state)
+        o = torch.empty((M, nv), dtype=torch.float32, device=dev)
+        K.gated_delta_scan(c[:, :nk], c[:, nk:2 * nk], c[:, 2 * nk:], proj[:, C + nv:C + nv + H], proj[:, C + nv + H:C + nv + 2 * H],
+                           self.a_log, self.dt_bias, self.unit_eps, dk ** -0.5, o, scan_state, step.cu_seqlens, step.seq_slots,
+                           H, H // G, dk, dv)
+        on = torch.empty((M, nv), dtype=dt, device=dev)
+        K.gated_norm(o, proj[:, C:C + nv], self.norm_w, self.eps, on, groups=H, gate_act="silu", gate_first=False)
+        linear(on, self.wo, residual, _out_mode)
+
+
 @register_mixer("parallel_mixers")
 class ParallelMixers(Mixer):
     """Two mixers side by side on the same input: left_scale * left(h) + right_scale * right(h).  At most one of
-    them caches keys and values; their per-sequence states lie one behind the other in the layer's state entry."""
+    them caches keys and values; their per-sequence states lie one behind the other in the layer's state entry.
+    ``out_norms`` {"left", "right": weight names, "size", "eps"}: each output is RMS-normed over the model's width, times its
+    own weight, before the factor; a block that can take the norms while it joins (``normed_ok``) is handed them undone."""
 
-    def __init__(self, runtime: Runtime, left, right, left_scale: float = 1.0, right_scale: float = 1.0):
+    def __init__(self, runtime: Runtime, left, right, left_scale: float = 1.0, right_scale: float = 1.0, out_norms: Optional[dict] = None):
         from .registry import build_part
         self.runtime = runtime
         self.left = build_part("mixer", left, runtime)
         self.right = build_part("mixer", right, runtime)
         self.scales = (float(left_scale), float(right_scale))
+        self.out_norms = dict(out_norms) if out_norms is not None else None
+        self.left_out = self.right_out = None
+        if self.out_norms is not None and not (hasattr(self.left, "forward_out") and hasattr(self.right, "forward_out")):
+            raise ValueError("mixers whose outputs are normed must return them (forward_out)")
         if self.left.kv_need() is not None and self.right.kv_need() is not None:
             raise ValueError("two mixers side by side that both cache keys and values are not built")
         sizes = [m.state_need().nbytes if m.state_need() is not None else 0 for m in (self.left, self.right)]
@@ -361,6 +513,12 @@ class ParallelMixers(Mixer):
 
     def sub_parts(self):
         return {"left": self.left, "right": self.right}
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        if self.out_norms is None:
+            return {}
+        n = self.out_norms
+        return {f"{side}_out": ParamSpec((ParamSource(n[side], (n["size"],)),), role="vector", init="ones") for side in ("left", "right")}
 
     def kv_need(self):
         return self.left.kv_need() or self.right.kv_need()
@@ -376,7 +534,24 @@ class ParallelMixers(Mixer):
             out.append(replace(cache, state=cache.state[:, at:at + n] if n else None))
         return out
 
-    def forward_out(self, xn, step, cache):
+    offers_normed = True       # ``forward_out(..., normed_ok=True)`` may return ``NormedTerm``s
+
+    def _normed_terms(self, xn, step, cache):
+        terms = []
+        for m, view, s, w in zip((self.left, self.right), self._views(cache), self.scales, (self.left_out, self.right_out)):
+            (y, f), = m.forward_out(xn, step, view)
+            if f != 1.0:
+                raise K.KernelError("a factor under an output norm is not built")
+            terms.append((NormedTerm(y, w, self.out_norms["eps"]), s))
+        return terms
+
+    def forward_out(self, xn, step, cache, normed_ok: bool = False):
+        if self.out_norms is not None:
+            if normed_ok:
+                return self._normed_terms(xn, step, cache)
+            y = torch.zeros((xn.shape[0], xn.shape[1]), dtype=torch.float32, device=xn.device)
+            self.forward(xn, y, step, cache)
+            return [(y, 1.0)]
         terms = []
         for m, view, s in zip((self.left, self.right), self._views(cache), self.scales):
             if hasattr(m, "forward_out"):
@@ -388,6 +563,10 @@ class ParallelMixers(Mixer):
         return terms
 
     def forward(self, xn, residual: torch.Tensor, step, cache):
+        if self.out_norms is not None:
+            K.branch_join(residual, 1.0, [K.JoinTerm(t.y, f, norm_weight=t.weight, eps=t.eps)
+                                          for t, f in self._normed_terms(xn, step, cache)])
+            return
         if self.scales != (1.0, 1.0):
             # the two outputs as tensors of their own, then residual += a * left + b * right in one pass
             terms = self.forward_out(xn, step, cache)

@@ -90,6 +90,7 @@ class HyperConnectedBlock(Block):
         return specs
 
     folds_norms = True
+    norm_requests = (StreamRead,)
 
     def _read(self, q: int) -> Optional[StreamRead]:
         norm = self.mixer_norm if q == 1 else self.feed_forward_norm
@@ -109,6 +110,8 @@ class HyperConnectedBlock(Block):
             y, factor = acc, 1.0
         kw = {}
         if not torch.is_tensor(y):                       # experts' rows, still unweighted (parts/moe.py, ExpertRows)
+            if y.weights is None:
+                raise K.KernelError("experts' rows that were weighed on their input: not built into the join of several streams")
             kw.update(row=y.row, weights=y.weights)
             y = y.rows
         else:
