@@ -69,6 +69,15 @@ __device__ __forceinline__ float rl_warp_max(float v) {
 // kernel launched the ordinary way both are no-ops.
 __device__ __forceinline__ void rl_pdl_trigger() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 __device__ __forceinline__ void rl_pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+// A pointer to what an earlier kernel of the step wrote, as seen behind the wait: p = rl_behind_wait(p).  To the compiler,
+// memory behind a `__restrict__` parameter is touched by nobody else, so the wait's memory clobber does not keep it from
+// loading through such a parameter before the wait; through the value that leaves this statement it cannot (volatile
+// statements keep their order).
+template <typename T>
+__device__ __forceinline__ T* rl_behind_wait(T* p) {
+  asm volatile("" : "+l"(p));
+  return p;
+}
 
 // 1 (default): launch with programmatic stream serialization; 0: ordinary launches
 // (rl_set_pdl, for measurements and for bisecting a fault).

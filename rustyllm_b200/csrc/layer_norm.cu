@@ -30,6 +30,7 @@ layer_norm_kernel(const float* __restrict__ x, const float* __restrict__ w0, con
   __shared__ float s_part[LN_THREADS / 32];
   rl_pdl_trigger();
   rl_pdl_wait();
+  x = rl_behind_wait(x);
   const int r = blockIdx.x;
   const float* xr = x + (size_t)(rows ? rows[r] : r) * d;
   float s = 0.f;
@@ -56,6 +57,7 @@ layer_norm_vec_kernel(const float* __restrict__ x, const float* __restrict__ w0,
   __shared__ float s_part[LN_THREADS / 32];
   rl_pdl_trigger();
   rl_pdl_wait();
+  x = rl_behind_wait(x);
   const int r = blockIdx.x;
   const float4* xr = reinterpret_cast<const float4*>(x + (size_t)(rows ? rows[r] : r) * d);
   const int nv = d / 4;

@@ -74,6 +74,7 @@ moe_route_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ wr, con
   float* s_x = s_logit + ((E + 3) & ~3);
   rl_pdl_trigger();
   rl_pdl_wait();
+  x = rl_behind_wait(x);
   const int m = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   moe_logits(x, ldx, wr, bias, d, E, s_logit, s_x);
   if (warp != 0) return;
@@ -116,7 +117,7 @@ moe_select_kernel(const float* __restrict__ logits, int M, int E, int top, int* 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int m = blockIdx.x * (MOE_THREADS / 32) + warp;
   if (m >= M) return;
-  const float* z = logits + (size_t)m * E;
+  const float* z = rl_behind_wait(logits) + (size_t)m * E;
   float chosen = 0.f, first = 0.f;
   int chosen_id = 0;
   unsigned taken_lo = 0;                 // experts this lane has given away already, for E <= 1024: bit j = expert lane + 32 j
@@ -291,6 +292,7 @@ moe_route_sigmoid_kernel(const T* __restrict__ x, int ldx, const T* __restrict__
   float* s_x = s_logit + 4 * Ep;
   rl_pdl_trigger();
   rl_pdl_wait();
+  x = rl_behind_wait(x);
   moe_logits(x, ldx, wr, (const float*)nullptr, d, E, s_logit, s_x);
   if (threadIdx.x >= 32) return;
   const size_t m = blockIdx.x;
@@ -306,6 +308,7 @@ moe_select_sigmoid_kernel(const float* __restrict__ logits, int E, int top, cons
   const int Ep = (E + 3) & ~3;
   rl_pdl_trigger();
   rl_pdl_wait();
+  logits = rl_behind_wait(logits);
   const size_t m = blockIdx.x;
   for (int e = threadIdx.x; e < E; e += 32) s_logit[e] = logits[m * E + e];
   __syncwarp();
@@ -382,6 +385,9 @@ moe_gate_up_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ wgu, 
   extern __shared__ float s_x[];          // [d]
   rl_pdl_trigger();
   rl_pdl_wait();
+  x = rl_behind_wait(x);
+  ids = rl_behind_wait(ids);
+  in_weights = rl_behind_wait(in_weights);
   const int pair = blockIdx.y, m = pair / top;
   const int e = ids[pair];
   const T* xr = x + (size_t)m * ldx;
@@ -430,6 +436,10 @@ moe_down_kernel(const T* __restrict__ h, const T* __restrict__ wd, const int* __
                 const float* __restrict__ weights, int d, int F, int top, float* __restrict__ residual) {
   rl_pdl_trigger();
   rl_pdl_wait();
+  h = rl_behind_wait(h);
+  ids = rl_behind_wait(ids);
+  weights = rl_behind_wait(weights);
+  residual = rl_behind_wait(residual);
   const int m = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int r = blockIdx.x * (MOE_THREADS / 32) + warp;
@@ -518,6 +528,7 @@ moe_plan_kernel(const int* __restrict__ ids, int pairs, int E, int bt, int max_t
   int* s_first = s_plan + E;
   rl_pdl_trigger();
   rl_pdl_wait();
+  ids = rl_behind_wait(ids);
   for (int e = threadIdx.x; e < E; e += blockDim.x) s_count[e] = 0;
   for (int t = threadIdx.x; t < max_tiles; t += blockDim.x) tile_group[t] = -1;
   __syncthreads();
@@ -543,6 +554,9 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x, int ldx, 
                                   const float* __restrict__ in_weights, __nv_bfloat16* __restrict__ xs) {
   rl_pdl_trigger();
   rl_pdl_wait();
+  x = rl_behind_wait(x);
+  row = rl_behind_wait(row);
+  in_weights = rl_behind_wait(in_weights);
   const int p = blockIdx.x;
   const __nv_bfloat16* src = x + (size_t)(p / top) * ldx;
   __nv_bfloat16* dst = xs + (size_t)row[p] * d;
@@ -569,6 +583,10 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
                                    int top, int d, float* __restrict__ residual) {
   rl_pdl_trigger();
   rl_pdl_wait();
+  y = rl_behind_wait(y);
+  row = rl_behind_wait(row);
+  weights = rl_behind_wait(weights);
+  residual = rl_behind_wait(residual);
   const int m = blockIdx.x;
   // d is a multiple of 4 and all rows are 16-byte aligned: four columns a thread, the choices' rows read side by side
   for (int i = 4 * threadIdx.x; i < d; i += 4 * blockDim.x) {

@@ -214,6 +214,7 @@ rope_kv_write_bf16_halves_kernel(__nv_bfloat16* __restrict__ qkv, int ld, const 
   __shared__ float2 cs[128];                              // (cos, sin) of the token's rot / 2 <= 128 angles
   rl_pdl_trigger();
   rl_pdl_wait();
+  qkv = rl_behind_wait(qkv);
   const int m = blockIdx.x;
   const int pos = positions[m];
   __nv_bfloat16* row = qkv + (size_t)m * ld;
