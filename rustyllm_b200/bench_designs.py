@@ -1,4 +1,4 @@
-"""Prompt and single-token throughput of the Mosurax, Mogutar, Forilorn, Besuzen and Buketar designs beside the Llama decoder at equal layer sizes
+"""Prompt and single-token throughput of the Mosurax, Mogutar, Forilorn, Besuzen, Buketar and Tigutar designs beside the Llama decoder at equal layer sizes
 (random bfloat16 weights, synthetic tokens): ``python bench.py --designs`` or
 ``python -m rustyllm_b200.bench_designs [--size NAME] [--steps K] [--warmup W]``.
 
@@ -26,6 +26,12 @@ uses together with the shared one are as wide as the dense feed-forward), vocabu
                  in as many parts as heads, one in four attention through a latent (1/4 of the width, at most 512, plus a
                  rotary key part of 64, queries straight from the input, a gate an element); every feed-forward 16
                  experts, 4 a token, each a quarter of the dense width, sigmoid scores, clamped gates
+  tigutar        layers of one layer norm that mixer and feed-forward both read; in four layers one of windowed attention (keys of
+                 half the head size, values of the whole) beside gated linear attention (heads of half x whole), one of the
+                 delta rule (heads of the head size, half as many query/key heads), and two of attention with a learned sink and
+                 a gate a head, the second on the first one's keys; feed-forwards in turn dense and 16 experts, 3 a token,
+                 each reading its score times the input
+``--tigutar-kernels`` times the Tigutar design's kernels alone, each beside the like kernel of the closest designs.
 ``--buketar-kernels`` times the Buketar design's kernels alone, each beside the like kernel of the closest designs.
 ``--besuzen-kernels`` times the Besuzen design's kernels alone, each beside the like kernel of the closest designs.
 ``--kernels`` times the Mogutar design's own kernels alone at the sizes of a layer (a JSON line a kernel, with the
@@ -50,7 +56,7 @@ SIZES = {
                   experts=16, top=3, expert_ff=3584, shared_ff=3584),
 }
 MAX_POSITIONS = 4096
-MODELS = ("llama", "mosurax-dense", "mosurax-moe", "mogutar", "forilorn", "besuzen", "buketar")
+MODELS = ("llama", "mosurax-dense", "mosurax-moe", "mogutar", "forilorn", "besuzen", "buketar", "tigutar")
 
 
 def llama_config(s: dict) -> dict:
@@ -136,6 +142,27 @@ def buketar_config(s: dict, streams: int = 4) -> dict:
             "layers": layers}
 
 
+def tigutar_config(s: dict, window: int = 1024) -> dict:
+    d, H, G, hd = s["width"], s["heads"], s["kv_heads"], s["dim"]
+    rot = {"base": 1.0e6, "dims": hd}
+    att = {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "rot": dict(rot)}
+    left = {"heads": H, "kv_heads": G, "dim": hd // 2, "vdim": hd, "scale": (hd // 2) ** -0.5, "rot": dict(rot, dims=hd // 2),
+            "mask": {"size": window}}
+    right = {"heads": d // hd, "dim": hd // 2, "vdim": hd, "tau": 16.0, "decay_rank": 16}
+    dense = {"kind": "dense", "ff": s["ff"]}
+    moe = {"kind": "moe", "router": {"experts": s["experts"], "top": s["top"]}, "expert": {"ff": s["expert_ff"], "limit": 7.0}}
+    layers = []
+    for i in range(s["layers"]):
+        mlp = dict(moe if i % 2 else dense)
+        if i % 4 == 0:
+            layers.append({"type": "parallel", "mixer": {"left": dict(left), "right": dict(right)}, "mlp": mlp})
+        elif i % 4 == 2:
+            layers.append({"type": "delta", "mixer": {"heads": d // hd, "kv_heads": d // hd // 2, "dim": hd, "vdim": hd, "conv": 4}, "mlp": mlp})
+        else:
+            layers.append({"type": "attention", "mixer": dict(att, kv_from=i - 2) if i % 4 == 3 else dict(att), "mlp": mlp})
+    return {"architecture": "Tigutar", "vocab": s["vocab"], "width": d, "norm": {"eps": 1e-5}, "residual_mult": 0.3, "layers": layers}
+
+
 def measure(config: dict, prompt: int, batches: List[int], context: int, steps: int, warmup: int) -> Dict[str, float]:
     import numpy as np
     import torch
@@ -197,7 +224,7 @@ def run(sizes: List[str], prompt: int = 2048, batches=(8, 64), context: int = 10
         s = SIZES[name]
         got = {}
         for model in models:
-            cfg = llama_config(s) if model == "llama" else buketar_config(s) if model == "buketar" else besuzen_config(s) if model == "besuzen" else mogutar_config(s, window or 1024) if model == "mogutar" \
+            cfg = tigutar_config(s, window or 1024) if model == "tigutar" else llama_config(s) if model == "llama" else buketar_config(s) if model == "buketar" else besuzen_config(s) if model == "besuzen" else mogutar_config(s, window or 1024) if model == "mogutar" \
                 else forilorn_config(s, window or 1024) if model == "forilorn" else mosurax_config(s, model == "mosurax-moe", window or None)
             got[model] = measure(cfg, prompt, list(batches), context, steps, warmup)
             line = {"size": name, "model": model, "prompt_tokens": prompt, "context": context, "window": window or None,
@@ -853,6 +880,155 @@ def buketar_kernel_times(sizes: List[str], prompt: int = 2048, batch: int = 64, 
     return t.lines
 
 
+def tigutar_kernel_times(sizes: List[str], prompt: int = 2048, batch: int = 64, context: int = 1024, window: int = 1024,
+                         runs: int = 20) -> List[dict]:
+    """The Tigutar design's kernels alone, each beside the like kernel of the closest designs (Besuzen: attention with a gate a
+    head, the recurrence with a decay a key channel, layer norms; Mogutar: the recurrence with a decay a head, the filter, the
+    norm that joins two mixers' outputs; Buketar: the join that sums experts' rows, the experts), bfloat16, at a layer's sizes:
+    ``prompt`` tokens of one sequence, and one token of each of ``batch`` sequences that hold ``context`` tokens with it."""
+    import torch
+    from . import kernels as K
+    from .cache.sequence_cache import KVNeed, SequenceCache
+    from .engine.step import StepState
+    t = _KernelTimer(runs)
+    dev, bf = t.dev, torch.bfloat16
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rnd = lambda *shape: torch.randn(shape, dtype=torch.float32, device=dev)
+    ones = lambda n: torch.ones(n, dtype=torch.float32, device=dev)
+
+    for name in sizes:
+        s = SIZES[name]
+        d, H, G, hd, E, F, top = s["width"], s["heads"], s["kv_heads"], s["dim"], s["experts"], s["expert_ff"], s["top"]
+        hk = hd // 2
+        for what, B, held, cnt in (("prompt", 1, 0, prompt), ("single tokens", batch, context - 1, 1)):
+            M = B * cnt
+            shape = f"{what}: {M} tokens, {B} seq of {held + cnt}"
+            cache = SequenceCache([KVNeed(G, hd), KVNeed(G, hk, window, hd)], [None, None], 64 * (-(-(held + cnt) // 64) + 1) * B, bf, dev, max_slots=B)
+            slots = [cache.alloc_slot() for _ in range(B)]
+            if held:
+                cache.prepare(slots, [held] * B); cache.commit(slots, [held] * B)
+            cache.prepare(slots, [cnt] * B)
+            st = StepState(M, B, i32([0] * M), i32([held + k for _ in range(B) for k in range(cnt)]),
+                           i32([sl for sl in slots for _ in range(cnt)]), i32([cnt * b for b in range(B + 1)]), i32(slots),
+                           i32([held + cnt] * B), i32([]), [cnt] * B, [held + cnt] * B, cnt, held + cnt, cnt == 1, length_spread=0)
+            (full, fl), (win, wl) = cache.kv_entry(0), cache.kv_entry(1)
+            kp, vp, kw, vw = full.k_pool(fl), full.v_pool(fl), win.k_pool(wl), win.v_pool(wl)
+            for pool in (kp, vp, kw, vw):
+                pool.normal_()
+            pairs = sum(p + 1 for p in range(held, held + cnt)) * B
+            wpairs = sum(min(p + 1, window) for p in range(held, held + cnt)) * B
+            # ---- attention ----
+            u, o = rnd(M, H * hd + H).to(bf), torch.empty((M, H * hd), dtype=bf, device=dev)
+            sinks, gate = rnd(H), u[:, H * hd:]
+            seen = (held + cnt) * B
+            for design, kwargs, label in (("tigutar", dict(sinks=sinks), "a sink's score and a gate a head"), ("besuzen", {}, "a gate a head")):
+                t.report(name, design, f"attention, {label}", f"{shape}, {H} heads over {G} of {hd}",
+                         lambda: K.attention(u, kp, vp, full.page_table, st, o, H, G, hd, hd ** -0.5, gate=gate, gate_per_head=True, **kwargs),
+                         seen * G * 2 * hd * 2 + 2 * M * H * hd * 2, 4.0 * pairs * H * hd)
+            uw = rnd(M, H * hk + G * (hk + hd)).to(bf)
+            t.report(name, "tigutar", f"attention, window {window}, keys of {hk}, values of {hd}", f"{shape}, {H} heads over {G}",
+                     lambda: K.attention(uw, kw, vw, win.page_table, st, o, H, G, hk, hk ** -0.5, window, value_dim=hd),
+                     min(seen, M + B * window) * G * (hk + hd) * 2 + M * H * (hk + hd) * 2, 2.0 * wpairs * H * (hk + hd))
+            t.report(name, "mosurax", f"attention, window {window}", f"{shape}, {H} heads over {G} of {hd}",
+                     lambda: K.attention(u, kp, vp, full.page_table, st, o, H, G, hd, hd ** -0.5, window),
+                     min(seen, M + B * window) * G * 2 * hd * 2 + 2 * M * H * hd * 2, 4.0 * wpairs * H * hd)
+            # ---- rotation and cache write ----
+            inv = torch.rand(hd // 2, dtype=torch.float32, device=dev)
+            ub = rnd(M, (H + 2 * G) * hd).to(bf)
+            t.report(name, "tigutar", f"rotation, keys of {hk} and values of {hd} to pages", f"{shape}, {H} + 2 x {G} heads",
+                     lambda: K.rope_kv_write(uw, st.positions, st.slot_of_token, win.page_table, inv, H, G, hk, hk, False, kw, vw, value_dim=hd),
+                     M * (2 * H * hk + 2 * G * (hk + hd)) * 2)
+            t.report(name, "tigutar", "rotation of queries alone", f"{shape}, {H} heads of {hd}",
+                     lambda: K.rope_kv_write(u, st.positions, st.slot_of_token, full.page_table, inv, H, 0, hd, hd, False, None, None),
+                     M * 2 * H * hd * 2)
+            t.report(name, "mosurax", "rotation, keys and values to pages", f"{shape}, {H} + 2 x {G} heads of {hd}",
+                     lambda: K.rope_kv_write(ub, st.positions, st.slot_of_token, full.page_table, inv, H, G, hd, hd, False, kp, vp),
+                     M * (2 * H + 4 * G) * hd * 2)
+            del cache, u, uw, ub, kp, vp, kw, vw, full, win
+            # ---- recurrences ----
+            Hr = d // hd
+            o32 = torch.empty((M, d), dtype=torch.float32, device=dev)
+            state = torch.zeros((B, 4 * Hr * hk * hd), dtype=torch.uint8, device=dev)
+            proj, z = rnd(M, 2 * Hr * hk + d).to(bf), rnd(M, Hr * hk)
+            nk = Hr * hk
+            moved = proj.numel() * 2 + z.numel() * 4 + o32.numel() * 4 + 2 * state.numel()
+            t.report(name, "tigutar", "gated linear attention, decay a key channel", f"{shape}, {Hr} heads of {hk} x {hd}",
+                     lambda: K.gated_linear_scan(proj[:, :nk], proj[:, nk:2 * nk], proj[:, 2 * nk:], z, 16.0, hk ** -0.5, o32, state, st.cu_seqlens,
+                                                 st.seq_slots, Hr, hk, hd), moved)
+            bonus = rnd(Hr, hk)
+            t.report(name, "besuzen", "recurrence, decay a key channel, bonus", f"{shape}, {Hr} heads of {hk} x {hd}",
+                     lambda: K.channel_decay_scan(proj[:, :nk], proj[:, nk:2 * nk], proj[:, 2 * nk:], z, bonus, o32, state, st.cu_seqlens, st.seq_slots,
+                                                  Hr, hk, hd), moved)
+            Gr = Hr // 2
+            state = torch.zeros((B, 4 * Hr * hd * hd), dtype=torch.uint8, device=dev)
+            c, ab, nk = rnd(M, 2 * Gr * hd + d).to(bf), rnd(M, 2 * Hr).to(bf), Gr * hd
+            zero = torch.zeros(Hr, dtype=torch.float32, device=dev)
+            t.report(name, "tigutar", "delta rule, decay a head", f"{shape}, {Hr} heads of {hd} x {hd}, {Gr} query/key heads",
+                     lambda: K.gated_delta_scan(c[:, :nk], c[:, nk:2 * nk], c[:, 2 * nk:], ab[:, :Hr], ab[:, Hr:], zero, zero, 1e-6, hd ** -0.5, o32, state,
+                                                st.cu_seqlens, st.seq_slots, Hr, 2, hd, hd), c.numel() * 2 + o32.numel() * 4 + 2 * state.numel())
+            t.report(name, "mogutar", "selective state space, decay a head", f"{shape}, {Hr} heads of {hd} x {hd}, {Gr} query/key heads",
+                     lambda: K.linear_scan(c[:, :nk], c[:, nk:2 * nk], c[:, 2 * nk:], o32, state, st.cu_seqlens, st.seq_slots, Hr, 2, hd, hd, zero,
+                                           dt_raw=ab[:, :Hr], dt_bias=zero), c.numel() * 2 + o32.numel() * 4 + 2 * state.numel())
+            # ---- the filter in front of the delta rule, the norm behind both ----
+            C = c.shape[1]
+            cw, cs, oc = rnd(C, 4), torch.zeros((B, 4 * 3 * C), dtype=torch.uint8, device=dev), torch.empty((M, C), dtype=bf, device=dev)
+            moved = 2 * M * C * 2 + 2 * cs.numel()
+            conv = lambda: (K.short_conv(c, cw, None, True, st.slot_of_token, cs, oc), K.short_conv_state(c, 4, st.cu_seqlens, st.seq_slots, cs))
+            t.report(name, "tigutar", "filter and its state", f"{shape}, {C} channels, 4 taps",
+                     conv if cnt > 1 else lambda: K.short_conv_step(c, cw, None, True, st.seq_slots, cs, oc), moved)
+            t.report(name, "mogutar", "short convolution + state", f"{shape}, {C} channels, 4 taps", conv, moved)
+            gt, on, wn = rnd(M, d).to(bf), torch.empty((M, d), dtype=bf, device=dev), ones(d)
+            t.report(name, "tigutar", "norm a head, weight, silu gate", f"{shape}, {Hr} heads of {hd}",
+                     lambda: K.gated_norm(o32, gt, wn, 1e-5, on, groups=Hr, gate_act="silu", gate_first=False), M * d * 8)
+            t.report(name, "besuzen", "norm a head, weight, silu gate", f"{shape}, {d // 64} heads of 64",
+                     lambda: K.gated_norm(o32, gt, wn, 1e-5, on, groups=d // 64, gate_act="silu", gate_first=False), M * d * 8)
+            # ---- the join ----
+            x, y0, y1, y2, w, bias, xb = rnd(M, d), rnd(M, d), rnd(M, d), rnd(M, d), ones(d), rnd(d), torch.empty((M, d), dtype=bf, device=dev)
+            two = [K.JoinTerm(y0, 0.5, norm_weight=w, eps=1e-5), K.JoinTerm(y1, 0.5, norm_weight=w, eps=1e-5), K.JoinTerm(y2)]
+            kwargs = dict(norm_weight=w, norm_bias=bias, norm_eps=1e-5, out=xb)
+            t.report(name, "tigutar", "two normed mixers and the feed-forward join, next norm", f"{shape}, width {d}",
+                     lambda: K.branch_join(x, 0.3, two, **kwargs), M * d * (3 * 4 + 8 + 2))
+            t.report(name, "mogutar", "stream += norm(a + b) w, rounded copy", f"{shape}, width {d}",
+                     lambda: K.norm_add(x, y0, 1.0, y1, 1.0, w, 1e-5, xb), M * d * (16 + 2))
+            rows, row = rnd(M * top, d), torch.randperm(M * top, device=dev).to(torch.int32)
+            exp = [K.JoinTerm(y0), K.JoinTerm(rows, row=row, top=top)]
+            t.report(name, "tigutar", f"a mixer and {top} experts' rows join, next norm", f"{shape}, width {d}",
+                     lambda: K.branch_join(x, 0.3, exp, **kwargs), M * d * (4 + 4 * top + 8 + 2))
+            X, wts = rnd(M, 1, d), torch.rand(M, top, device=dev)
+            mix, to, coef = ones(1).view(1, 1), ones(1), ones(1)
+            t.report(name, "buketar", f"one stream joined from {top} experts' rows, next normed read", f"{shape}, width {d}",
+                     lambda: K.streams_join(X, rows, mix, to, w, row=row, weights=wts, coef=coef, norm_weight=w, eps=1e-5, out=xb),
+                     M * d * (4 * top + 8 + 2))
+            t.report(name, "tigutar", "layer norm with a bias", f"{shape}, width {d}", lambda: K.layer_norm(x, w, xb, 1e-5, bias=bias), M * d * 6)
+            t.report(name, "besuzen", "layer norm", f"{shape}, width {d}", lambda: K.layer_norm(x, w, xb, 1e-5), M * d * 6)
+            del X, rows
+            # ---- router and experts ----
+            h, wr, logits = rnd(M, d).to(bf), (rnd(E, d) * d ** -0.5).to(bf), rnd(M, E)
+            ids, wt = torch.empty((M, top), dtype=torch.int32, device=dev), torch.empty((M, top), dtype=torch.float32, device=dev)
+            for design, grp, keep in (("tigutar", 1, 1), ("mogutar", 4, 2)):
+                kwargs = dict(softmax_all=False, group_top=2, renorm=False)
+                fn = (lambda: K.moe_route_scored(h, wr, None, top, grp, keep, ids, wt, **kwargs)) if M < 128 else \
+                    (lambda: K.moe_select_scored(logits, None, top, grp, keep, ids, wt, **kwargs))
+                t.report(name, design, ("router" if M < 128 else "choice from logits") + (", groups" if grp > 1 else ""), f"{shape}, {E} experts", fn,
+                         (M * d * 2 + E * d * 2) if M < 128 else M * E * 4 + M * top * 8)
+            wgu, wd = (rnd(E, F, 2, d) * d ** -0.5).to(bf), (rnd(E, d, F) * F ** -0.5).to(bf)
+            work = min(E, M * top) * 3 * F * d * 2 + M * top * (2 * d + 2 * F + F) * 2 + M * top * d * 4
+            for design, weigh in (("tigutar", True), ("buketar", False)):
+                t.report(name, design, "experts, clamped gate, weights on the " + ("input" if weigh else "output (in the join)"),
+                         f"{shape}, {top} of {E}, {d} x {F}",
+                         lambda: K.moe_experts_grouped(h, wgu, wd, ids, wt, None, act=(7.0, 1.702), weigh_input=weigh), work, 6.0 * M * top * F * d)
+            del wgu, wd
+            # ---- the decay's second projection ----
+            a2, b2, low, zz = (rnd(Hr * hk, 16)).to(bf), rnd(Hr * hk), rnd(M, 16).to(bf), torch.empty((M, Hr * hk), dtype=torch.float32, device=dev)
+            t.report(name, "tigutar", "decay's second projection, float out", f"{shape}, 16 -> {Hr * hk}",
+                     lambda: K.gemm_tc(low, a2, zz, K.OUT_F32, b2), M * (16 * 2 + Hr * hk * 4) + a2.numel() * 2, 2.0 * M * 16 * Hr * hk)
+            a2, b2, low, zz = (rnd(d, 64)).to(bf), rnd(d), rnd(M, 64).to(bf), torch.empty((M, d), dtype=torch.float32, device=dev)
+            t.report(name, "besuzen", "decay's second projection, float out", f"{shape}, 64 -> {d}",
+                     lambda: K.gemm_tc(low, a2, zz, K.OUT_F32, b2), M * (64 * 2 + d * 4) + a2.numel() * 2, 2.0 * M * 64 * d)
+    K.check_device_errors()
+    return t.lines
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("--size", action="append", choices=sorted(SIZES), help="default: all")
@@ -864,6 +1040,8 @@ def main(argv=None) -> int:
                     help="time the Besuzen design's kernels alone, each beside the like kernel of the Mosurax or Mogutar design, instead")
     ap.add_argument("--buketar-kernels", action="store_true",
                     help="time the Buketar design's kernels alone, each beside the like kernel of the closest designs, instead")
+    ap.add_argument("--tigutar-kernels", action="store_true",
+                    help="time the Tigutar design's kernels alone, each beside the like kernel of the closest designs, instead")
     ap.add_argument("--prompt", type=int, default=2048)
     ap.add_argument("--context", type=int, default=1024)
     ap.add_argument("--batch", type=int, action="append", help="default: 8 and 64")
@@ -879,6 +1057,9 @@ def main(argv=None) -> int:
         return 0
     if a.buketar_kernels:
         buketar_kernel_times(a.size or sorted(SIZES), a.prompt, max(a.batch or (64,)), a.context)
+        return 0
+    if a.tigutar_kernels:
+        tigutar_kernel_times(a.size or sorted(SIZES), a.prompt, max(a.batch or (64,)), a.context, a.window or 1024)
         return 0
     if a.kernels:
         kernel_times(a.size or sorted(SIZES), a.prompt, max(a.batch or (64,)))

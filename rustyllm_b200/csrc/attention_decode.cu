@@ -336,6 +336,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq, const __nv
   // ---- Q fragments (after the first key/value copies are on their way): rows = the m heads
   // of this KV head ----
   uint32_t qf[KS][4];
+  q = rl_behind_wait(q);
   {
     const __nv_bfloat16* q0 = q + (size_t)b * ldq + (size_t)(gkv * m + g) * HD + 2 * t;
     const __nv_bfloat16* q1 = q0 + (size_t)8 * HD;

@@ -228,4 +228,4 @@ def random_config(seed: int):
             layers.append(delta(G * pick(1, 2), G, pick(6, 8, 16, 33, 64), pick(8, 10, 24, 40), pick(1, 2, 3, 4, 6), rand_mlp()))
         else:
             layers.append(parallel(rand_att(True), pick(1, 2, 3), pick(6, 8, 16, 40), pick(8, 12, 24), pick(1.0, 4.0, 16.0), rand_mlp()))
-    return model(pick(31, 64, 150), d, pick(1e-5, 1e-6), pick(0.2, 0.5, 1.0), layers), pick(2, 4, 8)
+    return model(pick(31, 64, 150), d, pick(1e-5, 1e-6), pick(0.2, 0.35, 0.5), layers), pick(2, 4, 8)
