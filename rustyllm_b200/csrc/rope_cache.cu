@@ -205,7 +205,7 @@ rope_kv_write_bf16_pairs_kernel(__nv_bfloat16* __restrict__ qkv, int ld, const i
 
 // The same pairing where the general shape asks for more: a part of the head rotated (rotary width a multiple of 16), value
 // heads of another width, queries alone (G = 0, nothing cached).  A thread rotates eight pairs, or copies eight elements of
-// a key's unrotated tail or of a value; the token's sines and cosines once a CTA.
+// a key's unrotated tail or of a value; as many CTAs a token as it takes, the token's sines and cosines once a CTA.
 __global__ void __launch_bounds__(ROPE_THREADS)
 rope_kv_write_bf16_halves_kernel(__nv_bfloat16* __restrict__ qkv, int ld, const int* __restrict__ positions,
                                  const int* __restrict__ slot_of_token, const int* __restrict__ page_table, int max_pages,
@@ -233,7 +233,7 @@ rope_kv_write_bf16_halves_kernel(__nv_bfloat16* __restrict__ qkv, int ld, const 
   __syncthreads();
   const int pairs8 = half / 8, tail8 = (hd - rot) / 8, v8 = vd / 8;
   const int n_rot = (H + G) * pairs8, n_tail = G * tail8, n_v = G * v8;
-  for (int idx = threadIdx.x; idx < n_rot + n_tail + n_v; idx += ROPE_THREADS) {
+  for (int idx = blockIdx.y * ROPE_THREADS + threadIdx.x; idx < n_rot + n_tail + n_v; idx += gridDim.y * ROPE_THREADS) {
     if (idx < n_rot) {
       const int hs = idx / pairs8, i = (idx % pairs8) * 8;
       __nv_bfloat16* x = row + (size_t)hs * hd;
@@ -335,7 +335,9 @@ extern "C" int rl_rope_kv_write_mixed(void* qkv, int dtype, int ld, const int* p
   else if (v_other == nullptr && dtype == RL_BF16 && (write_cache || num_kv_heads == 0) && !interleaved && rotary_dim > 0 && rotary_dim % 16 == 0 &&
            head_dim % 8 == 0 && value_dim % 8 == 0 && ld % 8 == 0 && ((uintptr_t)qkv & 15) == 0 && ((uintptr_t)k_pool & 15) == 0 &&
            ((uintptr_t)v_pool & 15) == 0)
-    rl_launch_pdl(rope_kv_write_bf16_halves_kernel, dim3(num_tokens), threads, 0, stream, (__nv_bfloat16*)qkv, ld, positions, slot_of_token,
+    rl_launch_pdl(rope_kv_write_bf16_halves_kernel,
+                  dim3(num_tokens, ((num_heads + num_kv_heads) * rotary_dim / 16 + num_kv_heads * (head_dim - rotary_dim + value_dim) / 8 + threads - 1) / threads),
+                  threads, 0, stream, (__nv_bfloat16*)qkv, ld, positions, slot_of_token,
                   page_table, max_pages, inv_freq, num_heads, num_kv_heads, head_dim, value_dim, rotary_dim, (__nv_bfloat16*)k_pool,
                   (__nv_bfloat16*)v_pool);
   else if (dtype == RL_F32)
